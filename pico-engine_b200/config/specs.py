@@ -191,7 +191,9 @@ class GatedAttentionSpec(PartSpec):
     of a model that name the same ``value_blend_key`` share values: the "source" (the first of them in the schedule) uses and caches
     its own values and shows them to the others; a "reader" uses and caches (1 - l) v + l v_source, v_source the source's values of the
     same token and l its own stored number ``prefix + value_blend``.  ``position`` may also be a :class:`RotaryHalvesSpec`.
-    Tensor names are ``prefix + name``."""
+    ``qk_row_norm`` = (names of two weights behind the prefix): all query rows of a token together, and all its key rows together, are
+    RMS-normed (eps ``norm_eps``) with weights [n_heads * head_dim] and [n_kv_heads * head_dim] before ``position`` acts.  ``o_bias`` False:
+    with ``bias``, the output projection has none.  Tensor names are ``prefix + name``."""
     hidden: int
     n_heads: int
     n_kv_heads: int
@@ -218,6 +220,8 @@ class GatedAttentionSpec(PartSpec):
     value_blend: Optional[str] = None                        # tensor name (behind the prefix) of a reader's blending number
     value_blend_role: Optional[str] = None                   # "source", "reader" or None (values are the mixer's own business)
     value_blend_key: str = "values"
+    qk_row_norm: Optional[Tuple[str, str]] = None
+    o_bias: bool = True
 
 
 @dataclass(frozen=True)
@@ -292,7 +296,9 @@ class LinearAttentionSpec(PartSpec):
     ``decay_rank``.  ``qk_activation`` / ``v_activation`` ("none" or "silu") act on the projections, queries are
     multiplied by ``q_scale``.  The output is normed (RMS, eps ``norm_eps``, plain weight ``norm_name``) over all heads
     together (``norm_over`` "heads": weight of n_heads * v_head_dim) or head by head (``"head"``: one weight of
-    v_head_dim for all heads), multiplied by ``gate_activation`` ("sigmoid" or "silu") of W_g h, and projected by W_o."""
+    v_head_dim for all heads; ``norm_name`` None: no weight), multiplied by ``gate_activation`` ("sigmoid" or "silu") of W_g h, and
+    projected by W_o.  ``position`` (a :class:`RotaryPairsSpec` or :class:`RotaryHalvesSpec` without stretch; with a decay per head and
+    no activation of q and k) turns q and k, keys are then multiplied by ``k_scale``; both reach the recurrence in float32."""
     hidden: int
     n_heads: int
     head_dim: int
@@ -307,25 +313,29 @@ class LinearAttentionSpec(PartSpec):
     q_scale: float = 1.0
     norm_over: str = "heads"
     norm_eps: float = 1e-6
-    norm_name: str = "norm"
+    norm_name: Optional[str] = "norm"
     gate_activation: str = "sigmoid"
     q_name: str = "q"
     k_name: str = "k"
     v_name: str = "v"
     g_name: str = "g"
     o_name: str = "o"
+    position: Optional[PartSpec] = None
+    k_scale: float = 1.0
 
 
 @dataclass(frozen=True)
 class BranchSumSpec(PartSpec):
     """Several mixers side by side on the same input: the result is ``weight`` * sum_i rmsnorm(branch_i(h)) * w_i, each
-    branch's output normed over the model width (eps ``norm_eps``) with its own plain weight ``out_norms[i]``.  At most
-    one branch may keep keys and values; the branches' states lie one behind the other."""
+    branch's output normed over the model width (eps ``norm_eps``) with its own plain weight ``out_norms[i]``; or, with ``out_norms``
+    None, sum_i ``scales[i]`` * branch_i(h) without norms.  At most one branch may keep keys and values; the branches' states lie one
+    behind the other."""
     hidden: int
     branches: Tuple[PartSpec, ...]
-    out_norms: Tuple[str, ...]
+    out_norms: Optional[Tuple[str, ...]]
     norm_eps: float
     weight: float = 0.5
+    scales: Optional[Tuple[float, ...]] = None
 
 
 # ------------------------------------------------------------------ feed-forwards
@@ -354,7 +364,7 @@ class DenseMLPSpec(PartSpec):
 
 @dataclass(frozen=True)
 class GatedMLPSpec(PartSpec):
-    """down(act(gate(x)) * up(x)), no biases; ``activation`` "gelu_tanh" or "silu"; or "clamped_sigmoid": with g = min(gate(x), ``limit``)
+    """down(act(gate(x)) * up(x)), no biases; ``activation`` "gelu_tanh", "silu" or "relu"; or "clamped_sigmoid": with g = min(gate(x), ``limit``)
     and u = clamp(up(x), -``limit``, ``limit``) the hidden units are g * sigmoid(``alpha`` * g) * (u + 1).  Tensor names are ``prefix + name``."""
     hidden: int
     intermediate: int
@@ -415,7 +425,8 @@ class LayerSpec:
     x += scale1 * norm1(mixer(x)); x += scale2 * norm2(ffn(x)): the sublayers read the stream as it is and the norms
     act on their outputs (``mixer_scale`` / ``feed_forward_scale`` name the scale vectors; None: no scale); "sandwich" is
     x += out_norm1(mixer(norm1(x))); x += out_norm2(ffn(norm2(x))) with a norm before and one after each sublayer
-    (``mixer_out_norm`` / ``feed_forward_out_norm``).
+    (``mixer_out_norm`` / ``feed_forward_out_norm``); "streams" keeps several streams instead of one sum (``mixer_streams`` /
+    ``feed_forward_streams``, a :class:`StreamMixSpec` each).
     Every part is optional: a block without a feed-forward is a mixer-only block (pico-engine's
     recurrent layers are such, src/pico_engine/model.py:389-406), one without a mixer a feed-forward-only
     block, and a half without a norm takes the residual stream as it is.
@@ -432,6 +443,19 @@ class LayerSpec:
     feed_forward_scale: Optional[str] = None         # the same for the feed-forward
     mixer_out_norm: Optional[PartSpec] = None        # "sandwich": the norm of the mixer's output before it is added
     feed_forward_out_norm: Optional[PartSpec] = None  # the same for the feed-forward
+    mixer_streams: Optional[PartSpec] = None         # "streams": what the mixer reads of the streams and how its output enters them
+    feed_forward_streams: Optional[PartSpec] = None  # the same for the feed-forward
+
+
+@dataclass(frozen=True)
+class StreamMixSpec(PartSpec):
+    """A sublayer around a residual of ``streams`` streams x_1 .. x_s: it reads norm(u), u = sum_s in[s] x_s, and with y its output the
+    streams become x_t <- sum_s mix[s, t] x_s + out[t] y, all from the old ones.  ``in_name`` and ``out_name`` name vectors
+    [streams], ``mix_name`` a matrix [streams, streams] indexed [from, to]."""
+    streams: int
+    in_name: str
+    out_name: str
+    mix_name: str
 
 
 @dataclass(frozen=True)
@@ -473,12 +497,19 @@ class ModelPlan:
     stream_vectors: Tuple[Tuple[str, int], ...] = ()  # (tensor name, rows): [rows, hidden] tensors whose rows schedule entries add to the stream
     embedding_pairs: Optional[PartSpec] = None       # added to the embedding by (previous token, token) (a BigramTableSpec); None: nothing
     embedding_scale: float = 1.0                     # the embedded token is multiplied by this (the head reads the table as stored)
+    streams: Optional[int] = None                    # the residual is this many streams, all equal to the embedding at first; what leaves is their sum
 
     def validate(self) -> None:
         if not self.layers:
             raise ConfigError("a model needs at least one layer")
         if self.embedding_scale != 1.0 and self.embedding_pairs is not None:
             raise ConfigError("an embedding that reads pairs of tokens takes no scale")
+        for i, layer in enumerate(self.layers):
+            mixes = [m for m in (layer.mixer_streams, layer.feed_forward_streams) if m is not None]
+            if (layer.arrangement == "streams") != (self.streams is not None) or any(m.streams != self.streams for m in mixes):
+                raise ConfigError(f"layer {i}: its arrangement {layer.arrangement!r} does not fit a residual of {self.streams or 'no'} streams")
+        if self.streams is not None and any(e.add_embedding or e.add_vector is not None for e in self.schedule):
+            raise ConfigError("nothing is added between the layers of a residual of several streams")
         for e, entry in enumerate(self.schedule):
             if not 0 <= entry.layer < len(self.layers):
                 raise ConfigError(f"schedule[{e}] names layer {entry.layer}, but there are {len(self.layers)} layers")

@@ -2,18 +2,9 @@
 // every head and the cache write; a norm over groups of channels times a gate; the sum of several normed
 // branches into the residual stream; a scaled residual sum; vectors added to the stream; a gated activation
 // with a weight per group of columns; the choice of experts.
-#include "common.cuh"
+#include "activations.cuh"
 
 extern "C" void pe_set_pdl(int on) { pe_pdl_enabled() = on ? 1 : 0; }     // (this library's own copy of the switch)
-
-__device__ __forceinline__ float go_sigmoid(float v) { return 1.0f / (1.0f + expf(-v)); }
-__device__ __forceinline__ float go_gelu_tanh(float v) {
-    return 0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
-}
-// activations: 0 none, 1 sigmoid, 2 silu, 3 gelu (tanh form), 4 the square of relu
-__device__ __forceinline__ float go_act(float v, int act) {
-    return act == 1 ? go_sigmoid(v) : act == 2 ? v * go_sigmoid(v) : act == 3 ? go_gelu_tanh(v) : act == 4 ? (v > 0.f ? v * v : 0.f) : v;
-}
 
 // ---------------------------------------------------------------- rotation of pairs, unit norm, cache write
 // qkv [T, ld] in the step's dtype, a row = H*D query | G*D key | G*Dv value entries (| whatever else the product made).  In every query and key head the entries (2i, 2i+1), 2i+1 < rot_dims,
@@ -684,20 +675,7 @@ __global__ void gated_act_kernel(const T* gu, T* out, int I, int act, const floa
     }
 }
 
-// bfloat16, I a multiple of 8, aligned rows: eight columns a thread with 16-byte accesses.  Sigmoid and tanh come from the
-// special-function unit's 2^x and reciprocal (relative error about 2^-22, far below the bfloat16 rounding of the result).
-__device__ __forceinline__ float go_sigmoid_fast(float v) {
-    float e, r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-1.4426950408889634f * v));
-    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
-    return r;
-}
-__device__ __forceinline__ float go_act_fast(float v, int act) {
-    if (act == 2) return v * go_sigmoid_fast(v);
-    if (act == 3) return v * go_sigmoid_fast(1.5957691216057308f * (v + 0.044715f * v * v * v));   // 0.5 v (1 + tanh(u)) = v sigmoid(2u)
-    if (act == 1) return go_sigmoid_fast(v);
-    return v;
-}
+// bfloat16, I a multiple of 8, aligned rows: eight columns a thread with 16-byte accesses.
 __global__ void gated_act_bf16x8_kernel(const bf16* gu, bf16* out, int I, int act, const float* colw, int group, int n_groups, size_t units,
                                         float limit, float alpha) {
     pdl_launch_dependents();

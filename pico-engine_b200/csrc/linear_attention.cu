@@ -4,7 +4,8 @@
 //
 // a_t is either one constant per head (`head_decay` [H]) or one number per key channel and token,
 // a = sigmoid(z)^(inv_tau) = exp(-softplus(-z) * inv_tau) from float32 logits `z` [T, H*D].  q, k and v are columns of
-// `proj` [T, ld] (heads side by side, q_off / k_off / v_off the first column of each); an activation (0: none,
+// `proj` [T, ld] (heads side by side, q_off / k_off / v_off the first column of each), or, where q and k were worked on in
+// between and are float32 (`qk` [T, qk_ld]), q and k of those rows; an activation (0: none,
 // 1: silu) is applied to q and k and to v while they are loaded, and q is multiplied by `q_scale`.  Everything
 // after the load is float32; o [T, H*Dv] is written as float32.  A sequence's S lives in its slot of the state
 // area (`state` points at element 0 of slot 0, slots `state_stride` floats apart, [H, D, Dv] row-major) and is
@@ -34,6 +35,7 @@
 
 struct LAArgs {
     const void* proj; int ld, q_off, k_off, v_off;
+    const void* qk; int qk_ld;                 // the rows q and k are read from (proj itself, or float32 rows of their own)
     const void* z; int z_ld;
     const float* head_decay;
     float inv_tau, q_scale;
@@ -88,7 +90,7 @@ __device__ __forceinline__ void la_find_chunk(const int* row_first, const int* r
 // MODE 0: a sequence's tokens from its stored state; 1: a chunk from zero, leaving (A, L); 2: a chunk from its S_in.
 // NC: columns of the state a thread keeps (j and j + 32): with two, a block owns 64 columns, and every q, k and decay entry read
 // from shared memory meets two columns' multiply-adds.
-template <typename T, typename TZ, int R, int NC, bool PER_CHANNEL, int MODE>
+template <typename T, typename TQ, typename TZ, int R, int NC, bool PER_CHANNEL, int MODE>
 __global__ void __launch_bounds__(LA_THREADS) la_walk_kernel(LAArgs a) {
     pdl_launch_dependents();
     pdl_wait();
@@ -129,6 +131,7 @@ __global__ void __launch_bounds__(LA_THREADS) la_walk_kernel(LAArgs a) {
     const float hd = PER_CHANNEL ? 0.f : a.head_decay[h];
     float A = 1.f;                                       // MODE 1: the product of this chunk's decays on channel tid
     const T* proj = (const T*)a.proj;
+    const TQ* qk = (const TQ*)a.qk;
     const TZ* zp = (const TZ*)a.z;
 
     // A group's q, k, a and v are fetched into registers while the group before it is walked, and go to shared memory
@@ -142,8 +145,8 @@ __global__ void __launch_bounds__(LA_THREADS) la_walk_kernel(LAArgs a) {
             const int i = tid + n * LA_THREADS, tb = i / DP, d = i % DP;
             const size_t t = (size_t)(first + g0 + tb);
             const bool on = tb < ng && d < D;
-            fq[n] = on ? to_f(proj[t * a.ld + a.q_off + h * D + d]) : 0.f;
-            fk[n] = on ? to_f(proj[t * a.ld + a.k_off + h * D + d]) : 0.f;
+            fq[n] = on ? to_f(qk[t * a.qk_ld + a.q_off + h * D + d]) : 0.f;
+            fk[n] = on ? to_f(qk[t * a.qk_ld + a.k_off + h * D + d]) : 0.f;
             if constexpr (PER_CHANNEL) fa[n] = on ? to_f(zp[t * a.z_ld + h * D + d]) : 0.f;
         }
 #pragma unroll
@@ -268,31 +271,31 @@ __global__ void __launch_bounds__(256) la_carry_kernel(LAArgs a) {
     *sp = carry;
 }
 
-template <typename T, typename TZ, int R, int NC, bool PC>
+template <typename T, typename TQ, typename TZ, int R, int NC, bool PC>
 static int la_run(const LAArgs& a, int chunked, cudaStream_t s) {
     const int tiles = (a.Dv + LA_COLS * NC - 1) / (LA_COLS * NC);
     if (!chunked) {
-        PE_TRY(pe_launch(la_walk_kernel<T, TZ, R, NC, PC, 0>, dim3(a.B, a.H, tiles), LA_THREADS, 0, s, a));
+        PE_TRY(pe_launch(la_walk_kernel<T, TQ, TZ, R, NC, PC, 0>, dim3(a.B, a.H, tiles), LA_THREADS, 0, s, a));
         PE_LAUNCH_CHECK();
         return 0;
     }
-    PE_TRY(pe_launch(la_walk_kernel<T, TZ, R, NC, PC, 1>, dim3(a.max_chunks, a.H, tiles), LA_THREADS, 0, s, a));
+    PE_TRY(pe_launch(la_walk_kernel<T, TQ, TZ, R, NC, PC, 1>, dim3(a.max_chunks, a.H, tiles), LA_THREADS, 0, s, a));
     PE_LAUNCH_CHECK();
     const size_t per = (size_t)a.H * a.D * a.Dv;
     PE_TRY(pe_launch(la_carry_kernel, dim3((unsigned)((per + 255) / 256), a.B), 256, 0, s, a));
     PE_LAUNCH_CHECK();
-    PE_TRY(pe_launch(la_walk_kernel<T, TZ, R, NC, PC, 2>, dim3(a.max_chunks, a.H, tiles), LA_THREADS, 0, s, a));
+    PE_TRY(pe_launch(la_walk_kernel<T, TQ, TZ, R, NC, PC, 2>, dim3(a.max_chunks, a.H, tiles), LA_THREADS, 0, s, a));
     PE_LAUNCH_CHECK();
     return 0;
 }
 
 // Two columns a thread where the state is at least 64 columns wide and a thread's rows leave the registers for it.
-template <typename T, typename TZ, bool PC>
+template <typename T, typename TQ, typename TZ, bool PC>
 static int la_by_rows(const LAArgs& a, int chunked, cudaStream_t s) {
     const bool two = a.Dv >= 64;
-    if (a.D <= 8 * LA_DS) return two ? la_run<T, TZ, 8, 2, PC>(a, chunked, s) : la_run<T, TZ, 8, 1, PC>(a, chunked, s);
-    if (a.D <= 16 * LA_DS) return two ? la_run<T, TZ, 16, 2, PC>(a, chunked, s) : la_run<T, TZ, 16, 1, PC>(a, chunked, s);
-    if (a.D <= 32 * LA_DS) return la_run<T, TZ, 32, 1, PC>(a, chunked, s);
+    if (a.D <= 8 * LA_DS) return two ? la_run<T, TQ, TZ, 8, 2, PC>(a, chunked, s) : la_run<T, TQ, TZ, 8, 1, PC>(a, chunked, s);
+    if (a.D <= 16 * LA_DS) return two ? la_run<T, TQ, TZ, 16, 2, PC>(a, chunked, s) : la_run<T, TQ, TZ, 16, 1, PC>(a, chunked, s);
+    if (a.D <= 32 * LA_DS) return la_run<T, TQ, TZ, 32, 1, PC>(a, chunked, s);
     return PE_ERR_UNSUPPORTED;
 }
 
@@ -308,11 +311,12 @@ extern "C" int pe_linear_attention(const void* proj, int dtype, int ld, int q_of
                                    int z_ld, const float* head_decay, float inv_tau, float q_scale, int act_qk, int act_v,
                                    float* state, long long state_stride, const int* row_first, const int* row_lens,
                                    const int* slots, float* out, int T, int B, int H, int D, int Dv, int chunked, float* scratch,
-                                   void* stream) {
+                                   const float* qk, int qk_ld, void* stream) {
     if (T <= 0 || B <= 0) return 0;
     if ((z == nullptr) == (head_decay == nullptr) || D <= 0 || Dv <= 0 || H <= 0) return PE_ERR_UNSUPPORTED;
     if (chunked && !scratch) return PE_ERR_UNSUPPORTED;
     LAArgs a;
+    a.qk = qk ? (const void*)qk : proj; a.qk_ld = qk ? qk_ld : ld;
     a.proj = proj; a.ld = ld; a.q_off = q_off; a.k_off = k_off; a.v_off = v_off;
     a.z = z; a.z_ld = z_ld; a.head_decay = head_decay; a.inv_tau = inv_tau; a.q_scale = q_scale;
     a.act_qk = act_qk; a.act_v = act_v; a.state = state; a.state_stride = state_stride;
@@ -324,13 +328,13 @@ extern "C" int pe_linear_attention(const void* proj, int dtype, int ld, int q_of
     cudaStream_t s = (cudaStream_t)stream;
     const bool pc = z != nullptr;
     if (dtype == PE_F32) {
-        if (!pc) return la_by_rows<float, float, false>(a, chunked, s);
-        if (z_dtype == PE_F32) return la_by_rows<float, float, true>(a, chunked, s);
+        if (!pc) return la_by_rows<float, float, float, false>(a, chunked, s);
+        if (z_dtype == PE_F32) return la_by_rows<float, float, float, true>(a, chunked, s);
         return PE_ERR_UNSUPPORTED;
     }
     if (dtype == PE_BF16) {
-        if (!pc) return la_by_rows<bf16, bf16, false>(a, chunked, s);
-        if (z_dtype == PE_F32) return la_by_rows<bf16, float, true>(a, chunked, s);
+        if (!pc) return qk ? la_by_rows<bf16, float, float, false>(a, chunked, s) : la_by_rows<bf16, bf16, bf16, false>(a, chunked, s);
+        if (z_dtype == PE_F32 && !qk) return la_by_rows<bf16, bf16, float, true>(a, chunked, s);
     }
     return PE_ERR_UNSUPPORTED;
 }

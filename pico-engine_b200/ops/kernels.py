@@ -5,6 +5,7 @@ here with torch's allocator.  There is no other implementation behind these func
 from __future__ import annotations
 
 import os
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -949,23 +950,32 @@ def attention_headmix(q: torch.Tensor, q_stride: int, n_heads: int, n_kv: int, h
 # ---------------------------------------------------------------------------- gated mixers and routed feed-forwards
 
 LA_ACTIVATIONS = {"none": 0, "silu": 1}
-GATE_ACTIVATIONS = {"none": 0, "sigmoid": 1, "silu": 2, "gelu_tanh": 3, "relu2": 4, "clamped_sigmoid": 5}
+GATE_ACTIVATIONS = {"none": 0, "sigmoid": 1, "silu": 2, "gelu_tanh": 3, "relu2": 4, "clamped_sigmoid": 5, "relu": 6}
 
 
 def linear_attention(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, n_heads: int, head_dim: int, v_head_dim: int,
                      state: torch.Tensor, state_offset: int, row_first: torch.Tensor, row_lens: torch.Tensor, slots: torch.Tensor,
                      chunked: bool, head_decay: Optional[torch.Tensor] = None, decay_logits: Optional[torch.Tensor] = None,
                      inv_tau: float = 1.0, q_scale: float = 1.0, qk_activation: str = "none",
-                     v_activation: str = "none") -> torch.Tensor:
+                     v_activation: str = "none", qk: Optional[torch.Tensor] = None) -> torch.Tensor:
     """o [T, H * Dv] float32 of S_t = diag(a_t) S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head, for q, k, v at columns
     ``q_off``, ``k_off``, ``v_off`` of proj [T, ld] (packed sequences).  The decay is ``head_decay`` [H] float32 (one constant
     a head) or sigmoid(``decay_logits`` float32 [T, H * D])^``inv_tau`` (a number per key channel and token).  S [H, D, Dv] comes from
     and returns to the sequences' float32 state at ``state_offset``.  ``chunked``: prompts, three launches over chunks of
-    the sequences; else token after token in one launch."""
+    the sequences; else token after token in one launch.  ``qk`` (float32 [T, ld2], with a decay per head): q and k are the columns
+    ``q_off`` and ``k_off`` of these rows instead (rotated ones, that are not rounded on their way into the recurrence)."""
     T, ld = proj.shape
     H, D, Dv = n_heads, head_dim, v_head_dim
     _need(proj, "proj")
-    if max(q_off + H * D, k_off + H * D, v_off + H * Dv) > ld:
+    qk_ld = ld
+    if qk is not None:
+        _need(qk, "qk", torch.float32)
+        if qk.shape[0] != T:
+            raise KernelError("qk needs a row a token")
+        qk_ld = qk.shape[1]
+        if head_decay is None:
+            raise KernelError("queries and keys in rows of their own are taken with a decay per head")
+    if max(q_off + H * D, k_off + H * D) > qk_ld or v_off + H * Dv > ld:
         raise KernelError("q, k and v do not fit the rows of proj")
     if (head_decay is None) == (decay_logits is None):
         raise KernelError("linear attention takes either a decay per head or decay logits per channel")
@@ -985,7 +995,8 @@ def linear_attention(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, n_h
                                   0 if decay_logits is None else _code(decay_logits, "decay_logits"), H * D, _ptr(head_decay),
                                   float(inv_tau), float(q_scale), LA_ACTIVATIONS[qk_activation], LA_ACTIVATIONS[v_activation],
                                   sp, stride, row_first.data_ptr(), row_lens.data_ptr(), slots.data_ptr(), out.data_ptr(),
-                                  T, B, H, D, Dv, 1 if chunked else 0, ws, stream_ptr()), "linear_attention", 3 if chunked else 1)
+                                  T, B, H, D, Dv, 1 if chunked else 0, ws, _ptr(qk), qk_ld, stream_ptr()),
+          "linear_attention", 3 if chunked else 1)
     return out
 
 
@@ -1397,3 +1408,160 @@ def moe_route_stream_grouped(x: torch.Tensor, norm_weight: torch.Tensor, norm_bi
                                               _ptr(correction), 0 if correction is None else _code(correction, "correction"), n_groups, keep,
                                               group_best, float(factor), out.data_ptr(), _ptr(ids), T, stream_ptr()), "moe_route_stream_grouped")
     return out
+
+
+# ---------------------------------------------------------------------------- branches that share their first and last product
+
+@dataclass
+class NormedHeads:
+    """What ``heads_prepare`` does for an attention: the rows begin with H*D query, G*D key and G*Dv value entries.  All query entries of
+    a token are divided by their common root mean square and multiplied by ``q_weight`` [H*D], the key entries likewise with ``k_weight``
+    [G*D] (None: not normed); the first ``rot_dims`` entries of every head are turned by pos * freq[i], neighbours or (``halves``) entries
+    half of ``rot_dims`` apart; keys and values go to their cache pages (``k_pool`` None: they do not)."""
+    n_heads: int
+    n_kv: int
+    head_dim: int
+    v_head_dim: int
+    q_weight: Optional[torch.Tensor]
+    k_weight: Optional[torch.Tensor]
+    eps: float
+    freq: Optional[torch.Tensor]
+    rot_dims: int
+    halves: bool
+    k_pool: Optional[torch.Tensor] = None
+    v_pool: Optional[torch.Tensor] = None
+    block_table: Optional[torch.Tensor] = None
+    table_stride: int = 0
+
+
+@dataclass
+class TurnedHeads:
+    """What ``heads_prepare`` does for a linear attention: its queries (columns ``q_off`` ..) and keys (``k_off`` ..) turned as above,
+    the keys times ``k_scale``, as float32 rows [T, 2 * n_heads * head_dim] = queries | keys of their own."""
+    n_heads: int
+    head_dim: int
+    q_off: int
+    k_off: int
+    freq: Optional[torch.Tensor]
+    rot_dims: int
+    halves: bool
+    k_scale: float = 1.0
+
+
+def heads_prepare(proj: torch.Tensor, tok_pos: torch.Tensor, tok_row: torch.Tensor, normed: Optional[NormedHeads] = None,
+                  turned: Optional[TurnedHeads] = None) -> Optional[torch.Tensor]:
+    """One launch over the rows proj [T, ld] of a first product: ``normed`` in place, ``turned`` into new rows, which are returned."""
+    T, ld = proj.shape
+    _need(proj, "proj"); _need(tok_pos, "tok_pos", torch.int32, (T,)); _need(tok_row, "tok_row", torch.int32, (T,))
+    out = None
+    a, r = normed, turned
+    left = [0, 0, 0, 0, None, None, 0, 0.0, None, 0, 0, None, None, None, 0, 0]
+    if a is not None:
+        w_code = 0
+        for w, name, n in ((a.q_weight, "q_weight", a.n_heads * a.head_dim), (a.k_weight, "k_weight", a.n_kv * a.head_dim)):
+            if w is not None:
+                _need(w, name, None, (n,))
+                w_code = _code(w, name)
+        if a.q_weight is not None and a.k_weight is not None and a.q_weight.dtype != a.k_weight.dtype:
+            raise KernelError("the two norm weights must have one dtype")
+        if a.rot_dims:
+            _need(a.freq, "freq", torch.float32, (a.rot_dims // 2,))
+        store = a.k_pool is not None
+        if store:
+            _need(a.k_pool, "k_pool", proj.dtype); _need(a.v_pool, "v_pool", proj.dtype); _need(a.block_table, "block_table", torch.int32)
+            if tuple(a.k_pool.shape[1:]) != (a.n_kv, PAGE, a.head_dim) or tuple(a.v_pool.shape[1:]) != (a.n_kv, PAGE, a.v_head_dim):
+                raise KernelError(f"cache pools must be [pages, {a.n_kv}, {PAGE}, {a.head_dim}] and [pages, {a.n_kv}, {PAGE}, {a.v_head_dim}], "
+                                  f"not {tuple(a.k_pool.shape)} and {tuple(a.v_pool.shape)}")
+        left = [a.n_heads, a.n_kv, a.head_dim, a.v_head_dim, _ptr(a.q_weight), _ptr(a.k_weight), w_code, float(a.eps), _ptr(a.freq),
+                a.rot_dims, 1 if a.halves else 0, _ptr(a.k_pool), _ptr(a.v_pool), _ptr(a.block_table), a.table_stride, 1 if store else 0]
+    right = [0, 0, 0, 0, None, 0, 0, 0.0, None]
+    if r is not None:
+        if r.rot_dims:
+            _need(r.freq, "freq", torch.float32, (r.rot_dims // 2,))
+        out = torch.empty(T, 2 * r.n_heads * r.head_dim, dtype=torch.float32, device=proj.device)
+        right = [r.n_heads, r.head_dim, r.q_off, r.k_off, _ptr(r.freq), r.rot_dims, 1 if r.halves else 0, float(r.k_scale), out.data_ptr()]
+    check(gated().pe_heads_prepare(proj.data_ptr(), _code(proj, "proj"), ld, T, tok_pos.data_ptr(), tok_row.data_ptr(), *left, *right,
+                                   stream_ptr()), "heads_prepare")
+    return out
+
+
+@dataclass
+class GatedRows:
+    """One mixer's rows for ``gate_heads``: ``rows`` [T, C] float32 or the gate's dtype; ``group`` > 0: every run of so many channels is
+    divided by its root mean square and multiplied by ``weight`` [group] (None: ones); then times act(gate) with the gate at columns
+    ``gate_offset`` .. and times ``scale``."""
+    rows: torch.Tensor
+    group: int
+    weight: Optional[torch.Tensor]
+    eps: float
+    gate_offset: int
+    activation: str
+    scale: float
+
+
+def gate_heads(jobs, gate: torch.Tensor, width: int) -> torch.Tensor:
+    """The gated rows of up to four mixers side by side, [T, width] in gate's dtype (columns behind the last mixer's are zeros)."""
+    import ctypes
+    n = len(jobs)
+    T = gate.shape[0]
+    _need(gate, "gate")
+    offs, at = [], 0
+    for j in jobs:
+        _need(j.rows, "rows")
+        if j.rows.shape[0] != T or j.rows.dtype not in (torch.float32, gate.dtype):
+            raise KernelError("a mixer's rows must be float32 or of the gate's dtype, one a token")
+        if j.weight is not None:
+            _need(j.weight, "weight", None, (j.group,))
+        offs.append(at)
+        at += j.rows.shape[1]
+    if not 1 <= n <= 4 or at > width:
+        raise KernelError(f"{n} mixers of {at} channels do not fit rows of {width}")
+    ints = lambda values: (ctypes.c_int * n)(*values)
+    floats = lambda values: (ctypes.c_float * n)(*values)
+    ptrs = lambda values: (ctypes.c_void_p * n)(*values)
+    out = torch.empty(T, width, dtype=gate.dtype, device=gate.device)
+    check(gated().pe_gate_heads(n, ptrs(j.rows.data_ptr() for j in jobs), ints(1 if j.rows.dtype == torch.float32 else 0 for j in jobs),
+                                ints(j.rows.shape[1] for j in jobs), ints(j.group for j in jobs), ptrs(_ptr(j.weight) for j in jobs),
+                                ints(0 if j.weight is None else _code(j.weight, "weight") for j in jobs), floats(j.eps for j in jobs),
+                                ints(j.gate_offset for j in jobs), ints(GATE_ACTIVATIONS[j.activation] for j in jobs),
+                                floats(j.scale for j in jobs), ints(offs), T, gate.data_ptr(), gate.shape[1], out.data_ptr(), width,
+                                _code(gate, "gate"), stream_ptr()), "gate_heads")
+    return out
+
+
+# ---------------------------------------------------------------------------- a residual of several streams
+
+MAX_STREAMS = 32      # SM_MAX_STREAMS of csrc/branch_ops.cu
+
+
+def stream_mix(src: torch.Tensor, n_streams: int, dst: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None,
+               mix: Optional[torch.Tensor] = None, out_weights: Optional[torch.Tensor] = None, in_weights: Optional[torch.Tensor] = None,
+               norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0, out_dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+    """``src``: streams [T, S, W] float32, or one matrix [T, W] that all S streams equal.  With ``y`` [T, W] (float32 or bfloat16):
+    x_t <- sum_s mix[s, t] x_s + out_weights[t] y, all from the old ones (``mix`` [S, S], ``out_weights`` [S], float32).  ``dst`` [T, S, W]
+    (it may be ``src``) receives the streams.  With ``out_dtype``: returns u = sum_s in_weights[s] x_s of the streams as they now stand
+    (None: their sum) as [T, W], RMS-normed with ``norm_weight`` [W] (None: not normed)."""
+    S = n_streams
+    _need(src, "src", torch.float32)
+    T, W = src.shape[0], src.shape[-1]
+    one = src.dim() == 2
+    if not one and src.shape[1] != S:
+        raise KernelError(f"src holds {src.shape[1]} streams, not {S}")
+    if not 1 <= S <= MAX_STREAMS:
+        raise KernelError(f"{S} streams are not taken: 1 to {MAX_STREAMS} are")
+    if dst is not None:
+        _need(dst, "dst", torch.float32, (T, S, W))
+        if one and dst.data_ptr() == src.data_ptr():
+            raise KernelError("one matrix cannot be rewritten as several streams in place")
+    if y is not None:
+        _need(y, "y", None, (T, W)); _need(mix, "mix", torch.float32, (S, S)); _need(out_weights, "out_weights", torch.float32, (S,))
+    if in_weights is not None:
+        _need(in_weights, "in_weights", torch.float32, (S,))
+    if norm_weight is not None:
+        _need(norm_weight, "norm_weight", None, (W,))
+    h = None if out_dtype is None else torch.empty(T, W, dtype=out_dtype, device=src.device)
+    check(gated().pe_stream_mix(src.data_ptr(), W if one else S * W, 0 if one else W, _ptr(dst), _ptr(y), 0 if y is None else _code(y, "y"),
+                                _ptr(mix) if y is not None else None, _ptr(out_weights) if y is not None else None, _ptr(in_weights),
+                                _ptr(norm_weight), 0 if norm_weight is None else _code(norm_weight, "norm_weight"), float(eps), _ptr(h),
+                                0 if h is None else _code(h, "h"), T, S, W, stream_ptr()), "stream_mix")
+    return h

@@ -22,8 +22,9 @@ EXTRA_SOURCES = ("linear_mma.cu", "linear_batch.cu", "gemm_splitk.cu")
 MIXER_SOURCES = ("layernorm_conv.cu", "attention_headmix.cu", "attention_headmix_mma.cu", "attention_headmix_flash.cu",
                  "gated_recurrence.cu")
 # The kernels of gated mixers and routed feed-forwards (the linear-attention recurrence, rotation of pairs with unit norm and
-# cache write, norms over groups of channels with a gate, sums of normed branches, gated activations, the choice of experts).
-GATED_SOURCES = ("linear_attention.cu", "gated_ops.cu")
+# cache write, norms over groups of channels with a gate, sums of normed branches, gated activations, the choice of experts;
+# branches that share their first and last product, and residuals of several streams).
+GATED_SOURCES = ("linear_attention.cu", "gated_ops.cu", "branch_ops.cu")
 # The kernels of the state-space mixer (short convolution with silu, the recurrence with a scalar decay, gate then norm) and of
 # attention over one low-rank row per position.
 STATE_SOURCES = ("state_space.cu", "latent_ops.cu")
@@ -68,7 +69,7 @@ _MIXER_SIGNATURES = {
 }
 
 _GATED_SIGNATURES = {
-    "pe_linear_attention": [P, I, I, I, I, I, P, I, I, P, F, F, I, I, P, LL, P, P, P, P, I, I, I, I, I, I, P, P],
+    "pe_linear_attention": [P, I, I, I, I, I, P, I, I, P, F, F, I, I, P, LL, P, P, P, P, I, I, I, I, I, I, P, P, I, P],
     "pe_rotary_norm_store": [P, I, I, I, I, I, I, I, P, I, I, F, P, P, P, P, P, I, I, P],
     "pe_gated_norm": [P, I, I, I, I, P, I, F, P, I, I, I, P, I, P],
     "pe_normed_sum_add": [P, P, P, P, P, I, P, P, P, P, I, I, I, I, F, F, P],
@@ -81,6 +82,9 @@ _GATED_SIGNATURES = {
     "pe_moe_route_stream_grouped": [P, P, I, P, I, F, P, I, I, I, P, I, I, I, I, F, P, P, I, P],
     "pe_rotary_half_store": [P, I, I, I, I, I, I, I, P, I, F, I, F, P, P, P, P, P, I, I, P, I, P, I, P],
     "pe_moe_route_stream": [P, P, I, F, P, I, I, I, I, P, P, I, I, F, P],
+    "pe_heads_prepare": [P, I, I, I, P, P, I, I, I, I, P, P, I, F, P, I, I, P, P, P, I, I, I, I, I, I, P, I, I, F, P, P],
+    "pe_gate_heads": [I, P, P, P, P, P, P, P, P, P, P, P, I, P, I, P, I, I, P],
+    "pe_stream_mix": [P, LL, LL, P, P, I, P, P, P, P, I, F, P, I, I, I, I, P],
 }
 
 _STATE_SIGNATURES = {

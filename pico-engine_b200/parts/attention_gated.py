@@ -9,7 +9,7 @@ import math
 from ..config.specs import ConfigError, GatedAttentionSpec, NoPositionSpec, RotaryHalvesSpec, RotaryPairsSpec
 from ..ops import kernels, linear
 from ..weights.loader import ParamSpec
-from .base import Mixer, first_product, last_product_into, normed_rows, register_mixer
+from .base import Mixer, SharedProducts, first_product, last_product_into, normed_rows, register_mixer
 
 
 def pair_frequencies(spec: RotaryPairsSpec, device) -> torch.Tensor:
@@ -39,7 +39,7 @@ def halves_frequencies(spec: RotaryHalvesSpec, device):
 
 
 @register_mixer(GatedAttentionSpec)
-class GatedAttention(Mixer):
+class GatedAttention(Mixer, SharedProducts):
     """One product for q, k, v and the gate; rotation of neighbouring pairs of q and k, unit norm of every head and the
     cache write in one kernel (csrc/gated_ops.cu); attention over the cache (the kernels of grouped attention where keys
     and values have one size that they take, else the float32-score kernels that take any two sizes); the heads times
@@ -59,6 +59,13 @@ class GatedAttention(Mixer):
             raise ConfigError("value_blend_role is \"source\", \"reader\" (with the name of its number) or None")
         if spec.value_blend_role is not None and not (spec.own_kv and isinstance(spec.position, RotaryHalvesSpec)):
             raise ConfigError("values are blended in the kernel that rotates halves, for a mixer with keys and values of its own")
+        if spec.qk_row_norm is not None:
+            if spec.qk_unit_norm or not spec.own_kv or spec.value_blend_role is not None:
+                raise ConfigError("a norm over all query and all key rows goes with keys and values of the mixer's own and no other norm or blend of them")
+            if isinstance(spec.position, RotaryHalvesSpec) and spec.position.stretch is not None:
+                raise ConfigError("the rotation behind a norm over all query and key rows is not stretched")
+            if getattr(spec.position, "dims", 0) % 2 or getattr(spec.position, "dims", 0) > spec.head_dim:
+                raise ConfigError(f"{spec.position.dims} rotated entries do not fit a head of {spec.head_dim}")
         if spec.head_dim > 256 or spec.v_head_dim > 256:
             raise ConfigError(f"head sizes {spec.head_dim}/{spec.v_head_dim} are not taken: up to 256 are")
         if spec.window is not None and spec.window <= 0:
@@ -68,7 +75,7 @@ class GatedAttention(Mixer):
             raise ConfigError(f"{len(spec.distance_slopes)} distance slopes for {spec.n_heads} heads")
         if spec.keep_first < 0 or (spec.keep_first and spec.window is None):
             raise ConfigError("keep_first belongs to a window and cannot be negative")
-        self.w_in = self.w_o = self.freq = self.b_in = self.b_o = self.slopes = self.sink = self.blend_weight = None
+        self.w_in = self.w_o = self.freq = self.b_in = self.b_o = self.slopes = self.sink = self.blend_weight = self.q_norm = self.k_norm = None
         self.magnitude = 1.0
         # the kernels of grouped attention take equal key and value sizes: any up to 256 in float32, multiples of 16 in bfloat16;
         # a distance bias and kept first keys are known to the kernels that take two sizes
@@ -94,7 +101,10 @@ class GatedAttention(Mixer):
             out[p + s.value_blend] = ParamSpec((), init="normal")
         if s.bias:
             out.update({p + n + s.bias_suffix: ParamSpec((rows[n],), init="normal") for n in self._in_names() if n != s.gate})
-            out[p + s.o_name + s.bias_suffix] = ParamSpec((s.hidden,), init="normal")
+            if s.o_bias:
+                out[p + s.o_name + s.bias_suffix] = ParamSpec((s.hidden,), init="normal")
+        if s.qk_row_norm is not None:
+            out.update({p + n: ParamSpec((size,), init="one_plus_normal") for n, size in zip(s.qk_row_norm, (q, k))})
         return out
 
     def take_tensors(self, get):
@@ -113,7 +123,11 @@ class GatedAttention(Mixer):
             if pad:
                 biases.append(torch.zeros(pad, dtype=like.dtype, device=like.device))
             self.b_in = torch.cat([b.to(like.dtype) for b in biases]).contiguous()
-            self.b_o = get(p + s.o_name + s.bias_suffix)
+            self.b_o = get(p + s.o_name + s.bias_suffix) if s.o_bias else None
+        if s.qk_row_norm is not None:
+            self.q_norm, self.k_norm = (get(p + n) for n in s.qk_row_norm)
+            if self.q_norm.dtype != self.k_norm.dtype:
+                self.q_norm, self.k_norm = self.q_norm.float(), self.k_norm.float()
         if s.distance_slopes is not None:
             self.slopes = torch.tensor(s.distance_slopes, dtype=torch.float32, device=self.device)
         if s.fixed_sink is not None:
@@ -132,14 +146,14 @@ class GatedAttention(Mixer):
         elif self.dtype == torch.bfloat16:
             for_head_dim(self.spec.head_dim)
         if isinstance(self.spec.position, RotaryPairsSpec):
-            self.freq = pair_frequencies(self.spec.position, self.device)
+            self.freq = pair_frequencies(self.spec.position, self.device) if self.spec.position.dims else None
         elif isinstance(self.spec.position, RotaryHalvesSpec):
             self.freq, self.magnitude = halves_frequencies(self.spec.position, self.device)
             if not self.spec.position.dims:
                 self.freq = None
 
     def weights(self):
-        return [t for t in (self.w_in, self.w_o, self.b_in, self.b_o, self.blend_weight) if t is not None]
+        return [t for t in (self.w_in, self.w_o, self.b_in, self.b_o, self.blend_weight, self.q_norm, self.k_norm) if t is not None]
 
     def cache_needs(self):
         s = self.spec
@@ -160,6 +174,10 @@ class GatedAttention(Mixer):
             proj = linear(h if h is not None else x_norm[1].forward(x_norm[0], ctx.dtype), self.w_in, self.b_in, out_dtype=ctx.dtype)
         else:
             proj = first_product(*normed_rows(h, x_norm, ctx, self.w_in), self.w_in, ctx)
+        if s.qk_row_norm is not None:
+            kernels.heads_prepare(proj, ctx.tok_pos, ctx.tok_row, normed=self.prepare_jobs(proj, 0, ctx, cache_entry, owns_cache)[0])
+            a = self.mixed_rows(proj, 0, None, ctx, cache_entry, owns_cache)
+            return a if s.gate is None else kernels.gate_heads([self.gate_job(a, 0, 1.0)], proj, a.shape[1])
         rot_dims = s.position.dims if isinstance(s.position, (RotaryPairsSpec, RotaryHalvesSpec)) else 0
         n_kv = s.n_kv_heads if s.own_kv else 0             # a row of proj then has no key and value entries
         if isinstance(s.position, RotaryHalvesSpec):
@@ -178,13 +196,7 @@ class GatedAttention(Mixer):
             kernels.rotary_norm_store(proj, s.n_heads, n_kv, s.head_dim, s.v_head_dim, self.freq, rot_dims, s.qk_unit_norm,
                                       s.norm_eps, ctx.tok_pos, ctx.tok_row, kv.k if owns_cache else None, kv.v if owns_cache else None,
                                       kv.table if owns_cache else None, kv.stride)
-        if self.plain_kernels:
-            a = kernels.attention(proj, proj.shape[1], s.n_heads, s.n_kv_heads, s.head_dim, kv.k, kv.v, kv.table, kv.stride,
-                                  ctx.tok_pos, ctx.tok_row, s.window, s.scale, ctx, own_rows_only=owns_cache)
-        else:
-            a = kernels.attention_headmix(proj, proj.shape[1], s.n_heads, s.n_kv_heads, s.head_dim, s.v_head_dim, kv.k, kv.v,
-                                          kv.table, kv.stride, ctx.tok_pos, ctx.tok_row, s.window, s.scale, self.sink, None, ctx,
-                                          slopes=self.slopes, keep_first=s.keep_first)
+        a = self.mixed_rows(proj, 0, None, ctx, cache_entry, owns_cache)
         if s.gate is None:
             return a
         return kernels.gated_norm(a, 0, None, s.norm_eps, proj, q_w + (k_w + v_w if s.own_kv else 0), "sigmoid", ctx.dtype)
@@ -197,3 +209,38 @@ class GatedAttention(Mixer):
             return False                                   # the fused sum has no place for a bias
         last_product_into(x, self.gated_heads(None, ctx, cache_entry, owns_cache, (x, norm)), self.w_o, scale, ctx)
         return True
+
+    # ---------------------------------------------------------------- beside another mixer on the same input
+    def can_share(self):
+        return self.spec.qk_row_norm is not None and self.spec.gate is not None and not (self.spec.bias and self.spec.o_bias)
+
+    def give_input(self):
+        w, b = self.w_in, self.b_in
+        self.w_in = self.b_in = None
+        return w, b
+
+    def give_output(self):
+        w, self.w_o = self.w_o, None
+        return w
+
+    def prepare_jobs(self, proj, col, ctx, cache_entry, owns_cache):
+        s = self.spec
+        if col or not owns_cache:
+            raise ConfigError("an attention's queries stand at the front of the rows, and it writes its own keys and values")
+        kv = ctx.kv(cache_entry)
+        return kernels.NormedHeads(s.n_heads, s.n_kv_heads, s.head_dim, s.v_head_dim, self.q_norm, self.k_norm, s.norm_eps, self.freq,
+                                   0 if self.freq is None else s.position.dims, isinstance(s.position, RotaryHalvesSpec),
+                                   kv.k, kv.v, kv.table, kv.stride), None
+
+    def mixed_rows(self, proj, col, turned, ctx, cache_entry, owns_cache):
+        s, kv = self.spec, ctx.kv(cache_entry)
+        if self.plain_kernels:
+            return kernels.attention(proj, proj.shape[1], s.n_heads, s.n_kv_heads, s.head_dim, kv.k, kv.v, kv.table, kv.stride,
+                                     ctx.tok_pos, ctx.tok_row, s.window, s.scale, ctx, own_rows_only=owns_cache)
+        return kernels.attention_headmix(proj, proj.shape[1], s.n_heads, s.n_kv_heads, s.head_dim, s.v_head_dim, kv.k, kv.v,
+                                         kv.table, kv.stride, ctx.tok_pos, ctx.tok_row, s.window, s.scale, self.sink, None, ctx,
+                                         slopes=self.slopes, keep_first=s.keep_first)
+
+    def gate_job(self, rows, col, scale):
+        q, k, v, _ = self._widths()
+        return kernels.GatedRows(rows, 0, None, self.spec.norm_eps, col + q + k + v, "sigmoid", scale)

@@ -82,6 +82,8 @@ class StepContext:
     scratch: Dict[str, torch.Tensor] = field(default_factory=dict)   # named buffers that live as long as the step
     pending: Optional[torch.Tensor] = None  # a product [T, hidden] that still has to be added to the residual stream
     pending_norm: Optional["Norm"] = None   # the norm that product passes on its way into the stream (None: it is added as it is)
+    pending_streams: Optional["Part"] = None  # how it enters a residual of several streams (a StreamMix)
+    stream_source: Optional[torch.Tensor] = None  # the one matrix [T, hidden] that all streams still equal, before the first sum into them
 
     # A part whose product comes out of the library may leave the sum into the residual stream pending, so
     # that the norm that follows does both in one pass.  Whoever reads the stream first settles it: parts
@@ -100,6 +102,9 @@ class StepContext:
     def settle(self, x: torch.Tensor) -> None:
         if self.pending is not None:
             from ..ops import kernels
+            if self.pending_streams is not None:
+                self._mix_streams(x, dst=x)
+                return
             y, n = self.pending, self.pending_norm
             self.pending = self.pending_norm = None
             if n is None:
@@ -116,6 +121,30 @@ class StepContext:
         if n is None:
             return norm.add_forward(x, y.contiguous(), self.dtype)
         return n.add_into(x, y.contiguous(), then=norm, out_dtype=self.dtype)
+
+    # A residual of several streams x [T, S, hidden]: a sublayer's output waits in the same place (``defer_streams``), and the pass that
+    # brings it into the streams also makes what the next sublayer reads (``streams_normed``) or, behind the last layer, their sum.
+    def defer_streams(self, x: torch.Tensor, y: torch.Tensor, mix: "Part") -> None:
+        self.settle(x)
+        self.pending, self.pending_streams = y.contiguous(), mix
+
+    def streams_normed(self, x: torch.Tensor, mix: "Part", norm: "Norm") -> torch.Tensor:
+        """norm(sum_s mix.in[s] x_s) in the step's dtype, after what is pending has entered the streams."""
+        return self._mix_streams(x, x if self.pending is not None else None, mix.in_weights, norm.weight, norm.eps, self.dtype)
+
+    def streams_sum(self, x: torch.Tensor) -> torch.Tensor:
+        """The sum of the streams [T, hidden] float32, with what is pending (the streams themselves are not brought up to date)."""
+        return self._mix_streams(x, None, out_dtype=torch.float32)
+
+    def _mix_streams(self, x, dst=None, in_weights=None, norm_weight=None, eps=0.0, out_dtype=None):
+        from ..ops import kernels
+        y, m = self.pending, self.pending_streams
+        self.pending = self.pending_streams = None
+        src = x if self.stream_source is None else self.stream_source
+        if dst is not None:
+            self.stream_source = None                      # from here on the streams stand in x
+        return kernels.stream_mix(src, x.shape[1], dst, y, None if m is None else m.mix, None if m is None else m.out_weights, in_weights,
+                                  norm_weight, eps, out_dtype)
 
     def kv(self, cache_entry: int) -> KVView:
         g = self.cache.group_of[cache_entry]
@@ -215,6 +244,33 @@ class Mixer(Part):
         """x += apply(norm(x)); parts override this to fuse the norm and the residual sum."""
         from ..ops import kernels
         kernels.residual_add(x, self.apply(norm.forward(x, ctx.dtype), ctx, entry, cache_entry, owns_cache).contiguous())
+
+
+class SharedProducts:
+    """What a mixer offers so that it can stand beside another one on the same input with one first and one last product for both
+    (``BranchSum`` without norms).  ``col`` is the first of the mixer's columns in the rows of the shared first product."""
+
+    def can_share(self) -> bool:
+        return False
+
+    def give_input(self):
+        """(weights, biases or None) of the first product, rows a multiple of 8; the mixer keeps none of its own after this."""
+        raise NotImplementedError
+
+    def give_output(self) -> torch.Tensor:
+        raise NotImplementedError
+
+    def prepare_jobs(self, proj, col: int, ctx, cache_entry: int, owns_cache: bool):
+        """(kernels.NormedHeads or None, kernels.TurnedHeads or None): what has to be done to this mixer's columns first."""
+        return None, None
+
+    def mixed_rows(self, proj, col: int, turned, ctx, cache_entry: int, owns_cache: bool) -> torch.Tensor:
+        """The heads' outputs, before norm and gate; ``turned``: the rows a TurnedHeads job made."""
+        raise NotImplementedError
+
+    def gate_job(self, rows, col: int, scale: float):
+        """kernels.GatedRows: norm, gate and the weight of this mixer."""
+        raise NotImplementedError
 
 
 class InputFilter(Part):

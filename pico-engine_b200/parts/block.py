@@ -3,6 +3,7 @@ absent) and the arrangement that runs them around the residual stream."""
 from __future__ import annotations
 
 from ..config.specs import ConfigError, LayerSpec
+from .streams import StreamMix
 from ..cache import CacheNeeds
 from ..weights.loader import ParamSpec
 from .base import ARRANGEMENTS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, Norm, Part, build_part, register_arrangement
@@ -71,6 +72,11 @@ class Layer:
         self.mixer_scale = None if spec.mixer_scale is None else ScaleVector(spec.mixer_scale, _hidden_of(spec), dtype, device)
         self.feed_forward_scale = None if spec.feed_forward_scale is None else \
             ScaleVector(spec.feed_forward_scale, _hidden_of(spec), dtype, device)
+        self.mixer_streams = None if spec.mixer_streams is None else StreamMix(spec.mixer_streams, dtype, device)
+        self.feed_forward_streams = None if spec.feed_forward_streams is None else StreamMix(spec.feed_forward_streams, dtype, device)
+        if spec.arrangement == "streams" and ((self.mixer is None) != (self.mixer_streams is None)
+                                              or (self.feed_forward is None) != (self.feed_forward_streams is None)):
+            raise ConfigError("the streams arrangement takes a stream mix for every sublayer there is")
         if (self.mixer_input is not None and self.mixer is None) or (self.feed_forward_input is not None and self.feed_forward is None):
             raise ConfigError("an input filter needs the sublayer whose input it filters")
         try:
@@ -82,7 +88,7 @@ class Layer:
         """The parts that are there (a stand-in for an absent norm has no tensors and is left out)."""
         return tuple(p for p in (self.mixer, self.mixer_norm, self.mixer_input, self.feed_forward, self.feed_forward_norm,
                                  self.feed_forward_input, self.mixer_scale, self.feed_forward_scale, self.mixer_out_norm,
-                                 self.feed_forward_out_norm)
+                                 self.feed_forward_out_norm, self.mixer_streams, self.feed_forward_streams)
                      if p is not None and not isinstance(p, PassThrough))
 
     def cache_needs(self):
@@ -223,3 +229,21 @@ def sandwich(layer: Layer, x, ctx, entry, cache_entry, owns_cache) -> None:
         if part is layer.feed_forward and getattr(part, "routes_from_stream", False):
             extra["x_norm"] = (x, norm)                      # a router may read the float32 stream through the norm itself
         ctx.defer_normed_add(x, part.apply(h, ctx, *where, **extra), out_norm)
+
+
+@register_arrangement("streams")
+def streams(layer: Layer, x, ctx, entry, cache_entry, owns_cache) -> None:
+    """Around several streams x [T, S, hidden]: a sublayer reads norm(sum_s in[s] x_s), and its output y enters all of them,
+    x_t <- sum_s mix[s, t] x_s + out[t] y.  A sublayer hands over the float32 sums of its last product where it can; its entry into the
+    streams is left pending, so that it and the sum and norm in front of the next sublayer are one kernel in float32."""
+    from .norm import RMSNorm
+    halves = ((layer.mixer, layer.mixer_norm, layer.mixer_streams, (entry, cache_entry, owns_cache)),
+              (layer.feed_forward, layer.feed_forward_norm, layer.feed_forward_streams, ()))
+    for part, norm, mix, where in halves:
+        if part is None:
+            continue
+        if type(norm) is not RMSNorm:
+            raise ConfigError("the streams arrangement takes an RMS norm in front of every sublayer")
+        h = ctx.streams_normed(x, mix, norm)
+        extra = {"out_dtype": x.dtype} if getattr(part, "takes_out_dtype", False) else {}
+        ctx.defer_streams(x, part.apply(h, ctx, *where, **extra), mix)

@@ -86,14 +86,14 @@ class DenseMLP(FeedForward):
 @register_feed_forward(GatedMLPSpec)
 class GatedMLP(FeedForward):
     """down(act(gate(h)) * up(h)) without biases, gate and up as one product on concatenated weights; act is gelu
-    (tanh formula) or silu, or the clamped form min(gate, l) sigmoid(a min(gate, l)) (clamp(up, -l, l) + 1); formed in float32."""
+    (tanh formula), silu or relu, or the clamped form min(gate, l) sigmoid(a min(gate, l)) (clamp(up, -l, l) + 1); formed in float32."""
 
     takes_out_dtype = True      # apply(..., out_dtype=) gives the product's float32 sums where the caller goes on in float32
 
     def __init__(self, spec: GatedMLPSpec, dtype, device):
         super().__init__(spec, dtype, device)
-        if spec.activation not in ("gelu_tanh", "silu", "clamped_sigmoid"):
-            raise ConfigError(f"activation {spec.activation!r} is not known; known: gelu_tanh, silu, clamped_sigmoid")
+        if spec.activation not in ("gelu_tanh", "silu", "relu", "clamped_sigmoid"):
+            raise ConfigError(f"activation {spec.activation!r} is not known; known: gelu_tanh, silu, relu, clamped_sigmoid")
         if spec.activation == "clamped_sigmoid" and not (spec.limit is not None and spec.limit > 0):
             raise ConfigError(f"the clamped activation needs a positive limit, found {spec.limit!r}")
         self.w_gate_up = self.w_down = None

@@ -76,7 +76,7 @@ class DecoderModel:
 
     # ------------------------------------------------------------------ a step
     def hidden(self, token_ids: torch.Tensor, ctx: StepContext) -> torch.Tensor:
-        """The residual stream [T, hidden] float32 after the last layer."""
+        """The residual stream (the sum of the streams, where there are several) [T, hidden] float32 after the last layer."""
         pairs = self.plan.embedding_pairs
         if pairs is None:
             x = kernels.embed(self.embedding, token_ids, scale=self.plan.embedding_scale)
@@ -86,6 +86,8 @@ class DecoderModel:
         if self.embedding_position is not None:
             self.embedding_position.add_to(x, ctx)
         x0 = x.clone() if self._keeps_embedding else None
+        if self.plan.streams is not None:                  # all streams equal the embedding until the first sublayer's output enters them
+            ctx.stream_source, x = x, torch.empty(x.shape[0], self.plan.streams, x.shape[1], dtype=x.dtype, device=x.device)
         for e, entry in enumerate(self.plan.schedule):
             cache_entry = e if entry.cache_of is None else entry.cache_of
             if entry.add_embedding or entry.add_vector is not None:
@@ -93,6 +95,8 @@ class DecoderModel:
                 vec = None if entry.add_vector is None else self.stream_vectors[entry.add_vector[0]][entry.add_vector[1]]
                 kernels.add_rows(x, x0 if entry.add_embedding else None, vec)
             self.layers[entry.layer].run(x, ctx, e, cache_entry, entry.cache_of is None)
+        if self.plan.streams is not None:
+            return ctx.streams_sum(x)
         ctx.settle(x)
         return x
 
