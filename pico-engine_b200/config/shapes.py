@@ -134,9 +134,38 @@ SHAPES.update({
 })
 
 
+def lefilorn_shape(width: int, heads: int, kv_heads: int, dim: int, ff: int, layers: int, vocab: int, window: int = 1024, keep_first: int = 16,
+                   streams: int = 4, vdim: int | None = None, loop=None) -> dict:
+    """A Lefilorn config.json: every layer has windowed attention with kept first keys beside linear attention with a fixed decay (half as
+    many heads, three quarters of a head rotated), and a dense feed-forward; the residual is ``streams`` streams."""
+    right_heads = max(heads // 2, 1)
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim or dim, "scale": dim ** -0.5, "mask": {"size": window, "keep_first": keep_first},
+            "rot": {"base": 500000.0, "dims": dim}}
+    right = {"heads": right_heads, "dim": dim, "vdim": dim, "decay": [1.0 - 2.0 ** (-4.0 - 6.0 * h / right_heads) for h in range(right_heads)],
+             "rot": {"base": 10000.0, "dims": dim * 3 // 4 // 4 * 4}}
+    layer = {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 0.75, "right_scale": 0.5}, "mlp": {"kind": "dense", "ff": ff}}
+    d = {"architecture": "Lefilorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": float(width) ** 0.5},
+         "streams": streams, "layers": [layer for _ in range(layers)]}
+    if loop is not None:
+        d["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return d
+
+
+SHAPES.update({
+    "lefilorn-tiny": lefilorn_shape(64, 4, 2, 16, 160, 3, 256, window=40, keep_first=3, streams=2, loop=(1, 2, 2)),
+    "lefilorn-0.5b": lefilorn_shape(896, 14, 2, 64, 4864, 24, 151936),          # the widths of qwen2.5-0.5b
+    "lefilorn-7b": lefilorn_shape(3584, 28, 4, 128, 18944, 28, 152064),         # the widths of qwen2.5-7b
+})
+
+
 def with_layers(d: dict, n: int) -> dict:
-    """The shape with only its first ``n`` layers."""
+    """The shape with only its first ``n`` layers (a run of them that is repeated ends where they end)."""
     d = dict(d)
+    if isinstance(d.get("loop"), dict) and isinstance(d.get("layers"), list) and d["loop"].get("stop", 0) > n:
+        if d["loop"]["start"] >= n:
+            d.pop("loop")
+        else:
+            d["loop"] = dict(d["loop"], stop=n)
     if isinstance(d.get("layers"), list):
         d["layers"] = d["layers"][:n]
     else:

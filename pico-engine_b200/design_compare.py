@@ -6,11 +6,13 @@ distance bias and kept first keys, also on another layer's keys and values; late
 mixtures; a bigram embedding) or the Tenusun decoder (a layer norm before and after each sublayer; latent attention with a query
 row behind a sliding window; grouped attention with one added to the softmax denominator, stretched rotation of halves, blended values and an
 output gate; a clamped gated feed-forward; mixtures chosen by sigmoid scores among groups of experts; its kernels also beside Pupidra's like
-kernels) and the dense Qwen2 decoder, this library's closest other model.  Random weights; prefill and decode throughput of a few layers, and
+kernels) or the Lefilorn decoder (a residual of several streams; windowed attention with kept first keys and a norm over all query and all key
+rows beside rotated linear attention with a fixed decay, sharing their first and last product; a relu gated feed-forward; its kernels also
+beside Kevelorn's like kernels) and the dense Qwen2 decoder, this library's closest other model.  Random weights; prefill and decode throughput of a few layers, and
 the kernels of the new design each beside the Qwen2 kernel that does the like job, as fractions of the measured
 copy bandwidth or matrix throughput.
 
-    python -m pico_engine.design_compare [--design mebalorn|kevelorn|pupidra|tenusun] [--sizes s,m,l] [--tokens 2048] [--batch 8] [--context 2048] [--output FILE]
+    python -m pico_engine.design_compare [--design mebalorn|kevelorn|pupidra|tenusun|lefilorn] [--sizes s,m,l] [--tokens 2048] [--batch 8] [--context 2048] [--output FILE]
 """
 from __future__ import annotations
 
@@ -54,8 +56,16 @@ def tenusun_config(size: str, layers: int | None = None) -> dict:
     return tenusun_shape(W, H, G, D, F, layers or max(L, 4), VOCAB)          # four layers: both kinds of layer twice (the second attention blends values)
 
 
-DESIGNS = {"mebalorn": mebalorn_config, "kevelorn": kevelorn_config, "pupidra": pupidra_config, "tenusun": tenusun_config}
-FOUR_LAYERS = ("pupidra", "tenusun")
+def lefilorn_config(size: str, layers: int | None = None) -> dict:
+    from .config.shapes import lefilorn_shape
+    W, H, G, D, F, L = SIZES[size]
+    return lefilorn_shape(W, H, G, D, F, layers or max(L, 4), VOCAB)
+
+
+DESIGNS = {"mebalorn": mebalorn_config, "kevelorn": kevelorn_config, "pupidra": pupidra_config, "tenusun": tenusun_config,
+           "lefilorn": lefilorn_config}
+FOUR_LAYERS = ("pupidra", "tenusun", "lefilorn")
+BESIDE = {"tenusun": ("pupidra", pupidra_config), "lefilorn": ("kevelorn", lambda size: kevelorn_config(size, 4))}     # the closest other design
 
 
 def qwen2_config(size: str, layers: int | None = None) -> dict:
@@ -364,6 +374,50 @@ def tenusun_kernel_times(eng, size: str, tokens: int, batch: int, context: int, 
     B.close_sequences(eng, slots)
 
 
+def lefilorn_kernel_times(eng, size: str, tokens: int, batch: int, context: int, entry) -> None:
+    """The kernels of the Lefilorn parts at the sizes of this shape's layers (all layers are alike)."""
+    W, H, G, D, F, L = SIZES[size]
+    bf = torch.bfloat16
+    layer = eng.model.layers[0]
+    both = layer.mixer
+    att, ret = (both.branches[i] for i in both.order)
+    col = both.columns[1]
+    sa, sr = att.spec, ret.spec
+    RH, RD, RV, S = sr.n_heads, sr.head_dim, sr.v_head_dim, eng.model.plan.streams
+    out = entry.out
+    window, keep = sa.window, sa.keep_first
+
+    def calls(ctx, T, B, label, attention_size):
+        kv = ctx.kv(0)
+        proj = torch.randn(T, both.w_in.shape[0], device="cuda").to(bf)
+        normed, turned = att.prepare_jobs(proj, 0, ctx, 0, True)[0], ret.prepare_jobs(proj, col, ctx, 0, True)[1]
+        entry(f"{label} norm over all heads + rotation + cache write; rotation of the linear branch", device_us(lambda: kernels.heads_prepare(
+            proj, ctx.tok_pos, ctx.tok_row, normed, turned)), nbytes=T * ((H + 2 * G) * D * 2 * 2 + 2 * RH * RD * (2 + 4)))
+        entry(f"{label} attention (window, kept first keys)", device_us(lambda: att.mixed_rows(proj, 0, None, ctx, 0, True)), **attention_size)
+        qk = kernels.heads_prepare(proj, ctx.tok_pos, ctx.tok_row, None, turned)
+        us = device_us(lambda: ret.mixed_rows(proj, col, qk, ctx, 0, False))
+        entry(f"{label} recurrence, fixed decay, rotated float32 q and k", us,
+              nbytes=T * RH * (2 * RD * 4 + RV * (2 + 4)) + 2 * B * RH * RD * RV * 4)
+        out[f"{label} recurrence, fixed decay, rotated float32 q and k"]["float32_tflops_per_s"] = 4.0 * RH * RD * RV * T / us / 1e6
+        rows = [torch.randn(T, H * D, device="cuda").to(bf), torch.randn(T, RH * RV, device="cuda")]
+        entry(f"{label} both branches: norm per head, gates, factors", device_us(lambda: kernels.gate_heads(
+            [att.gate_job(rows[0], 0, 0.75), ret.gate_job(rows[1], col, 0.5)], proj, both.w_o.shape[1])), nbytes=T * (H * D * 2 * 3 + RH * RV * (4 + 2 + 2)))
+        x, y = torch.randn(T, S, W, device="cuda"), torch.randn(T, W, device="cuda")
+        m, n = layer.mixer_streams, layer.feed_forward_norm
+        entry(f"{label} output into the streams + what the next sublayer reads + norm", device_us(lambda: kernels.stream_mix(
+            x, S, x, y, m.mix, m.out_weights, m.in_weights, n.weight, n.eps, bf)), nbytes=T * W * (2 * S * 4 + 4 + 2))
+        gu = torch.randn(T, 2 * F, device="cuda").to(bf)
+        entry(f"{label} relu(gate) x up", device_us(lambda: kernels.gated_act(gu, "relu")), nbytes=T * F * 2 * 3)
+
+    slot, ctx = _prompt_context(eng, tokens)
+    seen = sum(min(p + 1, window + min(keep, max(0, p + 1 - window))) for p in range(tokens))
+    calls(ctx, tokens, 1, "prefill", dict(flops=4.0 * H * D * seen))
+    eng.cache.close(slot)
+    slots, ctx = _decode_context(eng, batch, context)
+    calls(ctx, batch, batch, "decode", dict(nbytes=batch * min(context, window + keep) * 2 * G * D * 2))
+    B.close_sequences(eng, slots)
+
+
 def kernel_times(size: str, tokens: int, batch: int, context: int, peaks: dict, design: str = "mebalorn") -> Dict[str, dict]:
     """Every kernel of the new design beside the like kernel of the Qwen2 decoder: microseconds, the bytes or
     multiply-adds it must move or do, and that as a fraction of the measured peak."""
@@ -384,18 +438,23 @@ def kernel_times(size: str, tokens: int, batch: int, context: int, peaks: dict, 
     # (the kernels of the Kevelorn parts are timed in a model of three layers, which has every kind of part once)
     first = kevelorn_config(size, 3) if design == "kevelorn" else DESIGNS[design](size)
     runs = [(design, first), ("qwen2", qwen2_config(size))]
-    if design == "tenusun":                                  # its kernels also beside the like kernels of Pupidra
-        runs.insert(1, ("pupidra beside", pupidra_config(size)))
+    if design in BESIDE:                                     # its kernels also beside the like kernels of the closest other design
+        other, other_config = BESIDE[design]
+        runs.insert(1, (other + " beside", kevelorn_config(size, 3) if other == "kevelorn" else other_config(size)))
     for design, cfg in runs:
-        if design in ("pupidra", "pupidra beside", "tenusun"):
+        if design in ("pupidra", "pupidra beside", "tenusun", "lefilorn", "kevelorn beside"):
             eng = Engine.from_config(config_from_dict(cfg), seed=1, draw_on="cuda", dtype="bfloat16")
             eng.ensure_cache(max(tokens, batch * context) + 64 * batch, max(tokens, context), max_seqs=batch + 1)
             if design == "tenusun":
                 tenusun_kernel_times(eng, size, tokens, batch, context, entry)
+            elif design == "lefilorn":
+                lefilorn_kernel_times(eng, size, tokens, batch, context, entry)
             elif design == "pupidra":
                 pupidra_kernel_times(eng, size, tokens, batch, context, entry)
+            elif design == "kevelorn beside":
+                kevelorn_kernel_times(eng, size, tokens, batch, context, _prefixed(entry, out, "kevelorn "))
             else:
-                pupidra_kernel_times(eng, size, tokens, batch, context, _prefixed(entry, out))
+                pupidra_kernel_times(eng, size, tokens, batch, context, _prefixed(entry, out, "pupidra "))
             kernels.check_status(eng.device)
             del eng
             torch.cuda.empty_cache()
@@ -468,31 +527,31 @@ def kernel_times(size: str, tokens: int, batch: int, context: int, peaks: dict, 
 
 
 class _prefixed:
-    """``entry`` under names that begin with "pupidra ": the like kernels of another design in the same record."""
+    """``entry`` under names that begin with ``prefix``: the like kernels of another design in the same record."""
 
-    def __init__(self, entry, out):
-        self.entry, self.out = entry, _PrefixedDict(out)
+    def __init__(self, entry, out, prefix):
+        self.entry, self.out, self.prefix = entry, _PrefixedDict(out, prefix), prefix
 
     def __call__(self, name, us, nbytes=None, flops=None):
-        self.entry("pupidra " + name, us, nbytes, flops)
+        self.entry(self.prefix + name, us, nbytes, flops)
 
 
 class _PrefixedDict:
-    def __init__(self, out):
-        self._out = out
+    def __init__(self, out, prefix):
+        self._out, self._prefix = out, prefix
 
     def __getitem__(self, name):
-        return self._out["pupidra " + name]
+        return self._out[self._prefix + name]
 
 
 def throughput(size: str, tokens: int, batch: int, context: int, steps: int = 64, design: str = "mebalorn") -> Dict[str, dict]:
-    """Prefill of one prompt and decode of ``batch`` sequences through the engines' own steps, both designs (for Tenusun also Pupidra)."""
+    """Prefill of one prompt and decode of ``batch`` sequences through the engines' own steps, both designs (and the closest other one, ``BESIDE``)."""
     from .engine.engine import Engine
     out = {}
     n_layers = max(SIZES[size][5], 4) if design in FOUR_LAYERS else None    # the same number of layers on both sides
     runs = [(design, DESIGNS[design](size)), ("qwen2", qwen2_config(size, n_layers))]
-    if design == "tenusun":
-        runs.insert(1, ("pupidra", pupidra_config(size)))
+    if design in BESIDE:
+        runs.insert(1, (BESIDE[design][0], BESIDE[design][1](size)))
     for design, cfg in runs:
         eng = Engine.from_config(config_from_dict(cfg), seed=1, draw_on="cuda", dtype="bfloat16")
         pre = B.prefill_device(eng, tokens)
