@@ -503,10 +503,10 @@ extern "C" int pe_stream_mix(const float* src, long long src_tok, long long src_
         const size_t smem = (size_t)W * 4;
         if (smem > 200 * 1024) return PE_ERR_UNSUPPORTED;
         if (h && h_dtype == PE_BF16) {
-            if (smem > 40 * 1024) PE_TRY(cudaFuncSetAttribute(stream_mix_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            PE_TRY(cudaFuncSetAttribute(stream_mix_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
             PE_TRY(pe_launch(stream_mix_kernel<bf16>, T, 256, smem, s, a));
         } else {
-            if (smem > 40 * 1024) PE_TRY(cudaFuncSetAttribute(stream_mix_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+            PE_TRY(cudaFuncSetAttribute(stream_mix_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
             PE_TRY(pe_launch(stream_mix_kernel<float>, T, 256, smem, s, a));
         }
     }

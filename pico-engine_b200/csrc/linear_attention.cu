@@ -23,68 +23,21 @@
 //    S_end = diag(A) S_in + L with A the product of the chunk's decays and L the chunk's own contribution, so
 //    pass 1 computes (A, L) of every chunk from S_in = 0, pass 2 walks a sequence's chunks in order (an element
 //    a thread), leaves each chunk's S_in where its L was and stores the sequence's new state, and pass 3 runs
-//    every chunk again from its S_in and writes the outputs.  Chunks never cross sequences: chunk c of the step
+//    every chunk again from its S_in and writes the outputs.  With a decay per head passes 1 and 3 are products of tiles
+//    (linear_attention_tiles.cu); with one per channel they walk a chunk's tokens.  Chunks never cross sequences: chunk c of the step
 //    is found from the rows' lengths on the device, so the grid depends on (T, B) only.
-#include "common.cuh"
+#include "linear_attention.cuh"
 
 #define LA_COLS 32
 #define LA_DS 8
 #define LA_THREADS (LA_COLS * LA_DS)
 #define LA_GROUP 8
-#define LA_CHUNK 64
-
-struct LAArgs {
-    const void* proj; int ld, q_off, k_off, v_off;
-    const void* qk; int qk_ld;                 // the rows q and k are read from (proj itself, or float32 rows of their own)
-    const void* z; int z_ld;
-    const float* head_decay;
-    float inv_tau, q_scale;
-    int act_qk, act_v;
-    float* state; long long state_stride;
-    const int* row_first; const int* row_lens; const int* slots;
-    float* out;
-    int B, H, D, Dv;
-    float* chunk_state;      // [chunks, H, D, Dv]
-    float* chunk_decay;      // [chunks, H, D]
-    int max_chunks;
-};
-
-// silu of a projection.  FAST (the bfloat16 engine, whose projections carry 8 bits): 2^x and the reciprocal from the
-// special-function unit, relative error about 2^-22; else the exact routines.  A block applies it to every q and k entry of
-// its head for each of its tokens, so its cost is paid once per 32 columns of the state.
-template <bool FAST>
-__device__ __forceinline__ float la_act(float v, int act) {
-    if (act != 1) return v;
-    if (FAST) {
-        float e, r;
-        asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-1.4426950408889634f * v));
-        asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
-        return v * r;
-    }
-    return v / (1.0f + expf(-v));
-}
 
 // a = sigmoid(z)^(inv_tau), through the logarithm: -softplus(-z) * inv_tau
 __device__ __forceinline__ float la_channel_decay(float z, float inv_tau) {
     const float u = -z;
     const float sp = fmaxf(u, 0.f) + log1pf(expf(-fabsf(u)));
     return expf(-sp * inv_tau);
-}
-
-// Which sequence chunk `c` of the step belongs to, its first packed token and its number of tokens (0: no such chunk).
-__device__ __forceinline__ void la_find_chunk(const int* row_first, const int* row_lens, int B, int c, int& row, int& first, int& count) {
-    int base = 0;
-    row = -1; first = 0; count = 0;
-    for (int b = 0; b < B; ++b) {
-        const int n = row_lens[b], nc = (n + LA_CHUNK - 1) / LA_CHUNK;
-        if (c < base + nc) {
-            const int local = c - base;
-            row = b; first = row_first[b] + local * LA_CHUNK;
-            count = min(LA_CHUNK, n - local * LA_CHUNK);
-            return;
-        }
-        base += nc;
-    }
 }
 
 // MODE 0: a sequence's tokens from its stored state; 1: a chunk from zero, leaving (A, L); 2: a chunk from its S_in.
@@ -279,14 +232,23 @@ static int la_run(const LAArgs& a, int chunked, cudaStream_t s) {
         PE_LAUNCH_CHECK();
         return 0;
     }
-    PE_TRY(pe_launch(la_walk_kernel<T, TQ, TZ, R, NC, PC, 1>, dim3(a.max_chunks, a.H, tiles), LA_THREADS, 0, s, a));
-    PE_LAUNCH_CHECK();
     const size_t per = (size_t)a.H * a.D * a.Dv;
-    PE_TRY(pe_launch(la_carry_kernel, dim3((unsigned)((per + 255) / 256), a.B), 256, 0, s, a));
-    PE_LAUNCH_CHECK();
-    PE_TRY(pe_launch(la_walk_kernel<T, TQ, TZ, R, NC, PC, 2>, dim3(a.max_chunks, a.H, tiles), LA_THREADS, 0, s, a));
-    PE_LAUNCH_CHECK();
-    return 0;
+    const dim3 carry((unsigned)((per + 255) / 256), a.B);
+    if constexpr (!PC) {
+        const int types = sizeof(T) == 4 ? 0 : sizeof(TQ) == 2 ? 1 : 2;
+        if (const int e = la_tiles_contributions(a, types, s)) return e;
+        PE_TRY(pe_launch(la_carry_kernel, carry, 256, 0, s, a));
+        PE_LAUNCH_CHECK();
+        return la_tiles_outputs(a, types, s);
+    } else {
+        PE_TRY(pe_launch(la_walk_kernel<T, TQ, TZ, R, NC, PC, 1>, dim3(a.max_chunks, a.H, tiles), LA_THREADS, 0, s, a));
+        PE_LAUNCH_CHECK();
+        PE_TRY(pe_launch(la_carry_kernel, carry, 256, 0, s, a));
+        PE_LAUNCH_CHECK();
+        PE_TRY(pe_launch(la_walk_kernel<T, TQ, TZ, R, NC, PC, 2>, dim3(a.max_chunks, a.H, tiles), LA_THREADS, 0, s, a));
+        PE_LAUNCH_CHECK();
+        return 0;
+    }
 }
 
 // Two columns a thread where the state is at least 64 columns wide and a thread's rows leave the registers for it.

@@ -24,7 +24,7 @@ MIXER_SOURCES = ("layernorm_conv.cu", "attention_headmix.cu", "attention_headmix
 # The kernels of gated mixers and routed feed-forwards (the linear-attention recurrence, rotation of pairs with unit norm and
 # cache write, norms over groups of channels with a gate, sums of normed branches, gated activations, the choice of experts;
 # branches that share their first and last product, and residuals of several streams).
-GATED_SOURCES = ("linear_attention.cu", "gated_ops.cu", "branch_ops.cu")
+GATED_SOURCES = ("linear_attention.cu", "linear_attention_tiles.cu", "gated_ops.cu", "branch_ops.cu")
 # The kernels of the state-space mixer (short convolution with silu, the recurrence with a scalar decay, gate then norm) and of
 # attention over one low-rank row per position.
 STATE_SOURCES = ("state_space.cu", "latent_ops.cu")

@@ -111,18 +111,21 @@ class LinearAttention(Mixer, SharedProducts):
     def mixed_rows(self, proj, col, turned, ctx, cache_entry, owns_cache, logits=None):
         s = self.spec
         qk, vo = self._sizes()
-        # Token after token, a block a (sequence, head, 32 columns of the state), unless that leaves the GPU empty: few sequences
-        # with many tokens run as three passes over chunks.  Measured on a B200 (16 heads of 128 x 128): one prompt of 2,048
-        # tokens 319 us in chunks against 709 us, four such prompts 1,985 us against 1,062 us.  (Either way gives the same
-        # numbers up to float32 rounding; rows that bring a few tokens, such as the idle rows of a padded step, do not count.)
-        long_rows = sum(1 for n in ctx.lens if n > 64)
-        blocks = long_rows * s.n_heads * ((s.v_head_dim + 31) // 32)
+        # With a decay per head, prompts run as products of tiles over chunks of 64 tokens; rows that bring a few tokens walk them.
+        # With a decay per channel a chunk is walked twice, which pays only where the walk would leave the GPU empty: token after token
+        # is a block a (sequence, head, 32 columns of the state).  Measured on a B200 (16 heads of 128 x 128): one prompt of 2,048
+        # tokens 319 us in chunks against 709 us, four such prompts 1,985 us against 1,062 us.  (Every way gives the same numbers up to
+        # float32 rounding; rows that bring a few tokens, such as the idle rows of a padded step, do not count.)
+        if self.head_decay is not None:
+            chunked = any(n > 16 for n in ctx.lens)
+        else:
+            chunked = 0 < sum(1 for n in ctx.lens if n > 64) * s.n_heads * ((s.v_head_dim + 31) // 32) < 192
         # (keys that are scaled but not turned: the scale moves to the queries, the output being linear in either)
         q_scale = s.q_scale if turned is not None else s.q_scale * s.k_scale
         first = 0 if turned is not None else col
         return kernels.linear_attention(proj, first, first + qk, col + 2 * qk, s.n_heads, s.head_dim, s.v_head_dim, ctx.state(cache_entry),
                                         self.state_offset, ctx.row_first, ctx.row_lens, ctx.slots,
-                                        chunked=0 < blocks < 192,
+                                        chunked=chunked,
                                         head_decay=self.head_decay, decay_logits=logits, inv_tau=1.0 / s.decay_tau,
                                         q_scale=q_scale, qk_activation=s.qk_activation, v_activation=s.v_activation, qk=turned)
 
