@@ -55,6 +55,20 @@ __global__ void __launch_bounds__(256) heads_prepare_kernel(HeadsArgs a) {
     const int job = blockIdx.y + (a.H > 0 ? 0 : 1);
     T* row = (T*)a.proj + (size_t)t * a.ld;
     const int pos = a.tok_pos[t];
+    // the row's entries are asked for before the angles are worked out
+    uint4 raw[VEC ? 4 : 1];
+    if constexpr (VEC) {
+        if (job == 0) {
+            const int units = (a.H + a.G) * a.D / 8;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int i = tid + e * nt;
+                raw[e] = i < units ? *reinterpret_cast<const uint4*>(row + i * 8) : make_uint4(0u, 0u, 0u, 0u);
+            }
+        }
+    }
+    long long page = -1;
+    if (job == 0 && a.store) page = a.table[(size_t)a.tok_row[t] * a.table_stride + pos / PE_PAGE];
     const float* freq = job == 0 ? a.freq : a.r_freq;
     const int half = (job == 0 ? a.rot : a.r_rot) / 2;
     for (int i = tid; i < half; i += nt) sincosf((float)pos * freq[i], &s_sin[i], &s_cos[i]);
@@ -65,6 +79,7 @@ __global__ void __launch_bounds__(256) heads_prepare_kernel(HeadsArgs a) {
         if (sizeof(T) == 2 && a.r_halves && half % 2 == 0 && D % 2 == 0 && a.r_q % 2 == 0 && a.r_k % 2 == 0 && a.ld % 2 == 0) {
             // two neighbouring pairs (or two neighbouring single entries) a thread: 4-byte reads, 8-byte writes
             const int per = (D - half) / 2, units = 2 * a.RH * per;
+#pragma unroll 2
             for (int i = tid; i < units; i += nt) {
                 const int h = i / per, u = 2 * (i - h * per);
                 const bool key = h >= a.RH;
@@ -101,20 +116,16 @@ __global__ void __launch_bounds__(256) heads_prepare_kernel(HeadsArgs a) {
         return;
     }
     const int D = a.D, nq = a.H * D, nk = a.G * D;
-    long long page = -1;
-    if (a.store) page = a.table[(size_t)a.tok_row[t] * a.table_stride + pos / PE_PAGE];
     const int in_page = pos % PE_PAGE;
     T* k_pool = (T*)a.k_pool;
     T* v_pool = (T*)a.v_pool;
     const bool store = a.store && page >= 0;
     if constexpr (VEC) {
-        uint4 raw[4];
         float sq = 0.f, sk = 0.f;
         const int units = (nq + nk) / 8;
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
             const int i = tid + e * nt;
-            raw[e] = i < units ? *reinterpret_cast<const uint4*>(row + i * 8) : make_uint4(0u, 0u, 0u, 0u);
             const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&raw[e]);
             float ss = 0.f;
 #pragma unroll

@@ -45,7 +45,7 @@ enum { GT_STORE = 0, GT_ACCUM = 1, GT_SWIGLU = 2, GT_ROPE = 3 };
 struct GtArgs {
     void* out; const void* bias; int bias_dtype;
     int M, N, K;           // M rows of A; N rows of W (SWIGLU: N = 2 I)
-    int I;                 // SWIGLU: columns of the result
+    int I, relu;           // SWIGLU: columns of the result; relu != 0: max(gate, 0) in place of silu
     int tiles_m, tiles;    // tiles along the rows of A; all tiles (tile t: m = t % tiles_m, n = t / tiles_m)
     // ROPE
     int n_q, n_kv, hd;
@@ -110,9 +110,10 @@ __device__ __forceinline__ unsigned gt_pack(float lo, float hi) {
     return *reinterpret_cast<unsigned*>(&v);
 }
 __device__ __forceinline__ float gt_round(float v) { return __bfloat162float(__float2bfloat16_rn(v)); }
-// silu(g) * u with g and u rounded to bfloat16 first, as the unfused path stores them
-__device__ __forceinline__ float gt_swiglu(float g, float u) {
+// silu(g) * u (relu != 0: max(g, 0) * u) with g and u rounded to bfloat16 first, as the unfused path stores them
+__device__ __forceinline__ float gt_swiglu(float g, float u, int relu) {
     g = gt_round(g); u = gt_round(u);
+    if (relu) return fmaxf(g, 0.f) * u;
     float e, r;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(-1.4426950408889634f * g));
     asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
@@ -223,7 +224,7 @@ __device__ __forceinline__ void gt_epilogue_tile(const GtArgs& p, const CUtensor
                             unsigned w[4];
 #pragma unroll
                             for (int e = 0; e < 4; ++e)
-                                w[e] = gt_pack(gt_swiglu(gate[i + 2 * e], up[i + 2 * e]), gt_swiglu(gate[i + 2 * e + 1], up[i + 2 * e + 1]));
+                                w[e] = gt_pack(gt_swiglu(gate[i + 2 * e], up[i + 2 * e], p.relu), gt_swiglu(gate[i + 2 * e + 1], up[i + 2 * e + 1], p.relu));
                             *reinterpret_cast<uint4*>(o + i) = make_uint4(w[0], w[1], w[2], w[3]);
                         }
                     }
@@ -303,7 +304,7 @@ __device__ __forceinline__ void gt_epilogue_tile(const GtArgs& p, const CUtensor
                 if (n < p.I) {
 #pragma unroll
                     for (int j = 0; j < 32; ++j)
-                        if (m0 + c + j < p.M) ((bf16*)p.out)[(size_t)(m0 + c + j) * p.I + n] = __float2bfloat16_rn(gt_swiglu(gate[j], up[j]));
+                        if (m0 + c + j < p.M) ((bf16*)p.out)[(size_t)(m0 + c + j) * p.I + n] = __float2bfloat16_rn(gt_swiglu(gate[j], up[j], p.relu));
                 }
             }
         } else if (EPI == GT_ROPE) {
@@ -763,14 +764,15 @@ static int gt_dispatch(const void* A, const void* W, GtArgs& p, int orientation,
 extern "C" int pe_gemm_tcgen05(const void* A, const void* W, const void* bias, int bias_dtype, void* out, int epilogue,
                                int M, int N, int K, int orientation, int* status, void* stream) {
     if (M <= 0 || N <= 0) return 0;
-    if (K <= 0 || K % 8 || N % 8 || epilogue < 0 || epilogue > 2 || orientation < 0 || orientation > 3 || !status) return PE_ERR_UNSUPPORTED;
+    if (K <= 0 || K % 8 || N % 8 || epilogue < 0 || epilogue > 3 || orientation < 0 || orientation > 3 || !status) return PE_ERR_UNSUPPORTED;
     if (((uintptr_t)A | (uintptr_t)W | (uintptr_t)out) & 15) return PE_ERR_UNSUPPORTED;
-    if (epilogue == 2 && (N % 16 || bias)) return PE_ERR_UNSUPPORTED;
+    if (epilogue >= 2 && (N % 16 || bias)) return PE_ERR_UNSUPPORTED;
     if (epilogue == 1 && bias) return PE_ERR_UNSUPPORTED;
     GtArgs p = {};
     p.out = out; p.bias = bias; p.bias_dtype = bias_dtype; p.M = M; p.N = N; p.K = K; p.I = N / 2;
     cudaStream_t s = (cudaStream_t)stream;
-    if (epilogue == 2) return gt_dispatch<GT_SWIGLU>(A, W, p, orientation, status, s);
+    p.relu = epilogue == 3;
+    if (epilogue >= 2) return gt_dispatch<GT_SWIGLU>(A, W, p, orientation, status, s);
     if (epilogue == 0) return gt_dispatch<GT_STORE>(A, W, p, orientation, status, s);
     return gt_dispatch<GT_ACCUM>(A, W, p, orientation, status, s);
 }

@@ -27,8 +27,13 @@ __device__ __forceinline__ float4 lt_act4(float4 v, int act, float scale) {
     if (act) { v.x = la_act<FAST>(v.x, act); v.y = la_act<FAST>(v.y, act); v.z = la_act<FAST>(v.z, act); v.w = la_act<FAST>(v.w, act); }
     return make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
 }
+// acc += a * b on four entries, two multiply-adds an instruction (fma.rn.f32x2: each half rounds as a plain one does)
 __device__ __forceinline__ void lt_fma4(float4& acc, float a, const float4& b) {
-    acc.x = fmaf(a, b.x, acc.x); acc.y = fmaf(a, b.y, acc.y); acc.z = fmaf(a, b.z, acc.z); acc.w = fmaf(a, b.w, acc.w);
+    asm("{\n\t.reg .b64 pa, b0, b1, c0, c1;\n\t"
+        "mov.b64 pa, {%4, %4};\n\tmov.b64 b0, {%5, %6};\n\tmov.b64 b1, {%7, %8};\n\tmov.b64 c0, {%0, %1};\n\tmov.b64 c1, {%2, %3};\n\t"
+        "fma.rn.f32x2 c0, pa, b0, c0;\n\tfma.rn.f32x2 c1, pa, b1, c1;\n\t"
+        "mov.b64 {%0, %1}, c0;\n\tmov.b64 {%2, %3}, c1;\n\t}"
+        : "+f"(acc.x), "+f"(acc.y), "+f"(acc.z), "+f"(acc.w) : "f"(a), "f"(b.x), "f"(b.y), "f"(b.z), "f"(b.w));
 }
 
 // pw[i] = a^i for i <= 64 (a^0 = 1, also for a = 0)

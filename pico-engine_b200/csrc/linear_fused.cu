@@ -59,7 +59,7 @@ struct LfArgs {
     int rows;                 // STORE/ACCUM: rows of W per CTA, 8 or 16
     int chunk, stages;        // columns per bulk copy (a multiple of 32) and copies in flight per row
     int ksplit, kc;           // STORE/ACCUM: ranges of K a tile is cut into (CTAs of a cluster) and columns per range
-    int I;                    // SWIGLU
+    int I, relu;              // SWIGLU; relu != 0: max(gate, 0) in silu's place
     // ROPE
     int n_q, n_kv, hd;
     const float* cos_t; const float* sin_t;
@@ -405,8 +405,8 @@ __global__ void __launch_bounds__(32 * LF_WARPS, LF_MIN_CTAS(NT, RT, EPI)) linea
             if (i < p.I) {
                 // the unfused path rounds gate and up to bfloat16 before the activation; so does this one
                 v_lo = __bfloat162float(__float2bfloat16_rn(v_lo)); v_hi = __bfloat162float(__float2bfloat16_rn(v_hi));
-                const float sig = 1.0f / (1.0f + expf(-v_lo));
-                ((bf16*)p.out)[(size_t)m * p.I + i] = __float2bfloat16_rn(v_lo * sig * v_hi);
+                const float act = p.relu ? fmaxf(v_lo, 0.f) : v_lo * (1.0f / (1.0f + expf(-v_lo)));
+                ((bf16*)p.out)[(size_t)m * p.I + i] = __float2bfloat16_rn(act * v_hi);
             }
         } else if (EPI == LF_ROPE) {
             const int half = p.hd >> 1, per_head = half >> 3;
@@ -598,6 +598,16 @@ extern "C" int pe_norm_gate_up_swiglu(const float* x, const void* norm_w, int no
     p.X = x; p.norm_w = norm_w; p.norm_w_dtype = norm_w_dtype; p.eps = eps; p.W = (const bf16*)W; p.out = act;
     p.M = M; p.N = 2 * I; p.K = K; p.I = I; p.rows = 16;
     return lf_launch<LF_RMSNORM, LF_SWIGLU>(p, I / 8, status, (cudaStream_t)stream);
+}
+
+// act[M, I] = f(a . Wg^T) * (a . Wu^T) of bfloat16 rows a [M <= 16, K]; f silu, or (relu != 0) max(., 0).
+extern "C" int pe_gate_up_act(const void* a, const void* W, void* act, int M, int I, int K, int relu, int* status, void* stream) {
+    if (M <= 0 || I <= 0) return 0;
+    if (M > 16 || K <= 0 || K % 8 || I % 8 || !lf_aligned(W) || !lf_aligned(a)) return PE_ERR_UNSUPPORTED;
+    LfArgs p = {};
+    p.A = (const bf16*)a; p.W = (const bf16*)W; p.out = act;
+    p.M = M; p.N = 2 * I; p.K = K; p.I = I; p.relu = relu; p.rows = 16;
+    return lf_launch<LF_PLAIN, LF_SWIGLU>(p, I / 8, status, (cudaStream_t)stream);
 }
 
 // q[M, n_q * hd] and the cache pages of keys and values from h = RMSNorm(x) (or from bfloat16

@@ -158,7 +158,7 @@ def kevelorn_kernel_times(eng, size: str, tokens: int, batch: int, context: int,
     def recurrences(ctx, T, B, chunked, label):
         proj = torch.randn(T, 4 * H * D, device="cuda").to(bf)
         z = torch.randn(T, H * D, device="cuda")
-        work = 4.0 * H * D * D * T * (2 if chunked else 1)        # multiply-adds x 2, and the chunked way walks every chunk twice
+        work = 4.0 * H * D * D * T                                # the recurrence's own multiply-adds x 2, however they are arranged
         moved = T * 4 * H * D * 2 + T * H * D * 4 + 2 * B * state_bytes
         us = device_us(lambda: kernels.linear_attention(proj, 0, H * D, 2 * H * D, H, D, D, ctx.state(e_fix), 0, ctx.row_first, ctx.row_lens,
                                                         ctx.slots, chunked, head_decay=fix.head_decay, qk_activation="silu", v_activation="silu"))

@@ -542,6 +542,17 @@ def norm_gate_up_swiglu(x: torch.Tensor, norm_weight: torch.Tensor, eps: float, 
     return act
 
 
+def gate_up_act(a: torch.Tensor, w_gate_up: torch.Tensor, activation: str = "silu") -> torch.Tensor:
+    """f(a Wg^T) * (a Wu^T) of bfloat16 rows a [M <= 16, K], w_gate_up [2I, K] (gate rows first); f "silu" or "relu"."""
+    M, K = a.shape
+    I = w_gate_up.shape[0] // 2
+    _need(a, "a", torch.bfloat16); _need(w_gate_up, "w_gate_up", torch.bfloat16, (2 * I, K))
+    act = torch.empty(M, I, dtype=torch.bfloat16, device=a.device)
+    check(core().pe_gate_up_act(a.data_ptr(), w_gate_up.data_ptr(), act.data_ptr(), M, I, K, {"silu": 0, "relu": 1}[activation],
+                                status_ptr(a.device), stream_ptr()), "gate_up_act")
+    return act
+
+
 def norm_qkv_rope_store(x: torch.Tensor, norm_weight: torch.Tensor, eps: float, w_qkv: torch.Tensor,
                         b_qkv: Optional[torch.Tensor], n_q: int, n_kv: int, head_dim: int, cos: Optional[torch.Tensor],
                         sin: Optional[torch.Tensor], tok_pos: torch.Tensor, tok_row: torch.Tensor,
@@ -593,11 +604,11 @@ def gemm_tcgen05_takes(a: torch.Tensor, w: torch.Tensor) -> bool:
 
 
 def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None,
-                 accumulate_into: Optional[torch.Tensor] = None, swiglu: bool = False,
+                 accumulate_into: Optional[torch.Tensor] = None, swiglu=False,
                  orientation: Optional[str] = None) -> torch.Tensor:
     """a [M, K] . w [N, K]^T on the tcgen05 tensor cores with a fused epilogue: bfloat16 result
     (+ bias); or added into the float32 tensor ``accumulate_into``; or, with ``swiglu`` and
-    w = [gate rows; up rows], silu(gate) * up as bfloat16 [M, N / 2].  ``orientation``: "rows" puts
+    w = [gate rows; up rows], silu(gate) * up (``swiglu`` "relu": max(gate, 0) * up) as bfloat16 [M, N / 2].  ``orientation``: "rows" puts
     the rows of ``a`` on the accumulator's lanes, "pairs" the same with 256 rows to a pair of CTAs
     (``cta_group::2``), "swapped" the rows of ``w`` (for up to a few hundred rows of ``a``); None
     chooses by M."""
@@ -610,9 +621,11 @@ def gemm_tcgen05(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] 
         _need(accumulate_into, "accumulate_into", torch.float32, (M, N))
         out, epilogue = accumulate_into, 1
     elif swiglu:
-        out, epilogue = torch.empty(M, N // 2, dtype=torch.bfloat16, device=a.device), 2
+        out, epilogue = torch.empty(M, N // 2, dtype=torch.bfloat16, device=a.device), 3 if swiglu == "relu" else 2
     else:
         out, epilogue = torch.empty(M, N, dtype=torch.bfloat16, device=a.device), 0
+    if orientation == "splitk" and epilogue == 3:
+        raise KernelError("the split-K product has no relu epilogue")
     if orientation == "splitk":                  # rows of w on the lanes, K cut over a cluster (up to 64 rows of a)
         check(extras().pe_gemm_splitk(a.data_ptr(), w.data_ptr(), _ptr(bias), 0 if bias is None else _code(bias, "bias"),
                                     out.data_ptr(), epilogue, M, N, K, status_ptr(a.device), stream_ptr()), "gemm_splitk")

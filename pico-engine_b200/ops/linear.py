@@ -172,20 +172,30 @@ def linear(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     return kernels.linear_simt(a, w, bias, out_dtype, accumulate_into)
 
 
-def gate_up_swiglu(h: torch.Tensor, w_gate_up: torch.Tensor) -> torch.Tensor:
-    """silu(h Wg^T) * (h Wu^T) [T, I] for h [T, K] and w_gate_up = [Wg; Wu] [2I, K]: one tcgen05 kernel with the
-    activation in its epilogue, or the product followed by the SwiGLU kernel."""
-    if h.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and _takes_tcgen05(h, w_gate_up) \
-            and w_gate_up.shape[0] % 16 == 0:
+def gate_up_act(h: torch.Tensor, w_gate_up: torch.Tensor, activation: str = "silu") -> torch.Tensor:
+    """f(h Wg^T) * (h Wu^T) [T, I] for h [T, K] and w_gate_up = [Wg; Wu] [2I, K], f silu or relu: in bfloat16 one fused decode product
+    (up to 16 rows, where the sizes allow) or one tcgen05 kernel with the activation in its epilogue, else the product followed by the
+    activation kernel."""
+    after = kernels.swiglu if activation == "silu" else (lambda y: kernels.gated_act(y, activation))
+    if h.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and w_gate_up.shape[0] % 16 == 0:
         M = h.shape[0]
-        key = ("swiglu", Choice.bucket(M), w_gate_up.shape[0], w_gate_up.shape[1])
-        if key not in Choice.table:
-            sh = _scratch_rows(Choice.bucket(M), h.shape[1], h.dtype, h.device)
-            Choice.pick(key, lambda: kernels.gemm_tcgen05(sh, w_gate_up, swiglu=True),
-                        lambda: kernels.swiglu(torch.mm(sh, w_gate_up.t())), launches_saved=1)
-        if Choice.table.get(key) == "tcgen05":
-            return kernels.gemm_tcgen05(h, w_gate_up, swiglu=True)
-    return kernels.swiglu(linear(h, w_gate_up, out_dtype=h.dtype))
+        if kernels.fused_takes(M, w_gate_up, h):
+            return kernels.gate_up_act(h, w_gate_up, activation)
+        if _takes_tcgen05(h, w_gate_up):
+            fused = True if activation == "silu" else activation
+            key = ("swiglu" if activation == "silu" else activation + "_gate", Choice.bucket(M), w_gate_up.shape[0], w_gate_up.shape[1])
+            if key not in Choice.table:
+                sh = _scratch_rows(Choice.bucket(M), h.shape[1], h.dtype, h.device)
+                Choice.pick(key, lambda: kernels.gemm_tcgen05(sh, w_gate_up, swiglu=fused), lambda: after(torch.mm(sh, w_gate_up.t())),
+                            launches_saved=1)
+            if Choice.table.get(key) == "tcgen05":
+                return kernels.gemm_tcgen05(h, w_gate_up, swiglu=fused)
+    return after(linear(h, w_gate_up, out_dtype=h.dtype))
+
+
+def gate_up_swiglu(h: torch.Tensor, w_gate_up: torch.Tensor) -> torch.Tensor:
+    """silu(h Wg^T) * (h Wu^T)."""
+    return gate_up_act(h, w_gate_up, "silu")
 
 
 def qkv_rope_store_takes(h: torch.Tensor, w_qkv: torch.Tensor, b_qkv: Optional[torch.Tensor], head_dim: int) -> bool:

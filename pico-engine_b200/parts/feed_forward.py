@@ -113,9 +113,9 @@ class GatedMLP(FeedForward):
         gated()                                            # build or load this part's kernels now, loudly
 
     def _activation(self, h, ctx, x_norm=None):
-        if self.spec.activation == "silu" and x_norm is None:
-            from ..ops.linear import gate_up_swiglu
-            return gate_up_swiglu(h, self.w_gate_up)
+        if self.spec.activation in ("silu", "relu") and x_norm is None:
+            from ..ops.linear import gate_up_act
+            return gate_up_act(h, self.w_gate_up, self.spec.activation)
         gate_up = first_product(*normed_rows(h, x_norm, ctx, self.w_gate_up), self.w_gate_up, ctx)
         return kernels.gated_act(gate_up, self.spec.activation, limit=self.spec.limit or 0.0, alpha=self.spec.alpha)
 

@@ -468,3 +468,35 @@ def test_relu_gate(dtype, I):
     got = kernels.gated_act(gu.cuda(), "relu").double().cpu()
     assert (got - want).abs().max() < (4e-2 if dtype == "bfloat16" else 1e-6)
     assert not got[gu[:, :I].double() < 0].any()
+
+
+@pytest.mark.parametrize("activation", ["relu", "silu"])
+@pytest.mark.parametrize("M,K,I", [(1, 64, 24), (3, 72, 100), (8, 896, 4864), (9, 200, 72), (16, 1024, 512)])
+def test_gate_up_and_activation_of_a_decode_step_in_one_kernel(activation, M, K, I):
+    from pico_engine.ops import kernels
+    from pico_engine.ops.linear import gate_up_act
+    g = torch.Generator().manual_seed(M * 10 + I)
+    h, w = torch.randn(M, K, generator=g).bfloat16(), (torch.randn(2 * I, K, generator=g) * K ** -0.5).bfloat16()
+    gate, up = h.double() @ w[:I].double().T, h.double() @ w[I:].double().T
+    want = (torch.clamp(gate, min=0) if activation == "relu" else gate * plain.sigmoid(gate)) * up
+    fused = I % 8 == 0
+    if fused:
+        got = kernels.gate_up_act(h.cuda(), w.cuda(), activation).double().cpu()
+        assert (got - want).abs().max() < 3e-2 * max(1.0, float(want.abs().max()))
+        if activation == "relu":
+            assert not got[gate < -0.05].any()
+    got = gate_up_act(h.cuda(), w.cuda(), activation).double().cpu()
+    assert got.shape == (M, I) and (got - want).abs().max() < 3e-2 * max(1.0, float(want.abs().max()))
+
+
+@pytest.mark.parametrize("orientation", ["rows", "swapped", "pairs"])
+@pytest.mark.parametrize("M,K,I", [(17, 128, 64), (100, 896, 304), (300, 200, 1000)])
+def test_relu_gate_in_the_epilogue_of_the_tcgen05_product(orientation, M, K, I):
+    from pico_engine.ops import kernels
+    g = torch.Generator().manual_seed(M + I)
+    h, w = torch.randn(M, K, generator=g).bfloat16(), (torch.randn(2 * I, K, generator=g) * K ** -0.5).bfloat16()
+    gate, up = h.double() @ w[:I].double().T, h.double() @ w[I:].double().T
+    got = kernels.gemm_tcgen05(h.cuda(), w.cuda(), swiglu="relu", orientation=orientation).double().cpu()
+    want = torch.clamp(gate, min=0) * up
+    assert (got - want).abs().max() < 3e-2 * max(1.0, float(want.abs().max()))
+    kernels.check_status(torch.device("cuda", 0))
