@@ -152,7 +152,7 @@ def lefilorn_shape(width: int, heads: int, kv_heads: int, dim: int, ff: int, lay
 
 
 SHAPES.update({
-    "lefilorn-tiny": lefilorn_shape(64, 4, 2, 16, 160, 3, 256, window=40, keep_first=3, streams=2, loop=(1, 2, 2)),
+    "lefilorn-tiny": lefilorn_shape(64, 4, 2, 16, 160, 3, 256, window=48, keep_first=3, streams=2, loop=(1, 2, 2)),
     "lefilorn-0.5b": lefilorn_shape(896, 14, 2, 64, 4864, 24, 151936),          # the widths of qwen2.5-0.5b
     "lefilorn-7b": lefilorn_shape(3584, 28, 4, 128, 18944, 28, 152064),         # the widths of qwen2.5-7b
 })
