@@ -2,7 +2,8 @@
 from .specs import (ConfigError, PartSpec, RMSNormSpec, LayerNormSpec, RotaryHalfSpec, NoPositionSpec, SinusoidAddSpec,
                     CausalConvAddSpec, GQAAttentionSpec, HeadMixAttentionSpec, MinGRUSpec, SwiGLUSpec, DenseMLPSpec,
                     LayerSpec, ScheduleEntry, ModelPlan, RotaryPairsSpec, GatedAttentionSpec, LinearAttentionSpec, BranchSumSpec,
-                    GatedMLPSpec, MixtureSpec, LatentAttentionSpec, StateSpaceSpec, BigramTableSpec, RotaryHalvesSpec, StreamMixSpec)
+                    GatedMLPSpec, MixtureSpec, LatentAttentionSpec, StateSpaceSpec, BigramTableSpec, RotaryHalvesSpec, StreamMixSpec,
+                    DifferentialAttentionSpec)
 from .registry import (Architecture, register_architecture, known_architectures, architecture,
                        architecture_name_of, config_from_dict, read_config)
 from .qwen2 import Qwen2Config
@@ -11,6 +12,7 @@ from .kevelorn import KevelornConfig
 from .pupidra import PupidraConfig
 from .tenusun import TenusunConfig
 from .lefilorn import LefilornConfig
+from .razelorn import RazelornConfig
 
 __all__ = ["ConfigError", "PartSpec", "RMSNormSpec", "LayerNormSpec", "RotaryHalfSpec", "NoPositionSpec",
            "SinusoidAddSpec", "CausalConvAddSpec", "GQAAttentionSpec", "HeadMixAttentionSpec", "MinGRUSpec",
@@ -18,4 +20,4 @@ __all__ = ["ConfigError", "PartSpec", "RMSNormSpec", "LayerNormSpec", "RotaryHal
            "known_architectures", "architecture", "architecture_name_of", "config_from_dict", "read_config",
            "Qwen2Config", "KevelornConfig", "RotaryPairsSpec", "GatedAttentionSpec", "LinearAttentionSpec", "BranchSumSpec",
            "GatedMLPSpec", "MixtureSpec", "LatentAttentionSpec", "StateSpaceSpec", "BigramTableSpec", "PupidraConfig", "RotaryHalvesSpec", "TenusunConfig",
-           "StreamMixSpec", "LefilornConfig"]
+           "StreamMixSpec", "LefilornConfig", "DifferentialAttentionSpec", "RazelornConfig"]

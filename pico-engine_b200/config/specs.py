@@ -76,12 +76,15 @@ class RotaryHalvesSpec(PartSpec):
     entries of the head stay as they are.  ``stretch`` = (factor, original, fast, slow) lengthens the slow turns: with
     where(t) = dims * ln(original / (2 pi t)) / (2 ln base), lo = max(floor(where(fast)), 0), hi = min(ceil(where(slow)), dims - 1)
     and ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) the frequency is f_i / factor * ramp_i + f_i * (1 - ramp_i), and cos
-    and sin are multiplied by ``magnitude_slope`` * ln(factor) + 1."""
+    and sin are multiplied by ``magnitude_slope`` * ln(factor) + 1.  ``bands`` = (factor, low, high, original) decides by the wavelength
+    l = 2 pi / f_i instead: below original / high the frequency stays, above original / low it is divided by the factor, and in between
+    it is (1 - s) f_i / factor + s f_i with s = (original / l - low) / (high - low); cos and sin are as they are."""
     head_dim: int
     dims: int
     base: float
     stretch: Optional[Tuple[float, float, float, float]] = None
     magnitude_slope: float = 0.1
+    bands: Optional[Tuple[float, float, float, float]] = None
 
 
 @dataclass(frozen=True)
@@ -259,6 +262,36 @@ class LatentAttentionSpec(PartSpec):
 
 
 @dataclass(frozen=True)
+class DifferentialAttentionSpec(PartSpec):
+    """Softmax attention with grouped key/value heads in which a head has two maps, each with a query and a key of ``head_dim`` entries
+    of its own, over the same values of ``v_head_dim``.  W_q h and W_k h are laid out head by head as [map 1 | map 2].  Every query
+    and key row of a map is RMS-normed over its entries (weights ``q_norm`` / ``k_norm`` [head_dim], shared by all heads and maps; None:
+    as projected; eps ``norm_eps``) and then turned by ``position`` (a :class:`RotaryHalvesSpec` without stretch, or none).  With a1 and
+    a2 the two maps' outputs and lambda = exp(sum(l1 * l2)) - exp(sum(l3 * l4)) + ``lambda_base`` (``lambda_names``: four vectors
+    [head_dim]) a head's output is (a1 - lambda a2) / sqrt(mean((a1 - lambda a2)^2) + norm_eps) * ``out_scale``; then W_o.  ``window``
+    as in :class:`GQAAttentionSpec`.  Tensor names are ``prefix + name``."""
+    hidden: int
+    n_heads: int
+    n_kv_heads: int
+    head_dim: int
+    v_head_dim: int
+    window: Optional[int]
+    scale: float
+    position: PartSpec
+    prefix: str
+    lambda_base: float
+    out_scale: float
+    norm_eps: float = 1e-6
+    q_norm: Optional[str] = "q.norm"
+    k_norm: Optional[str] = "k.norm"
+    lambda_names: Tuple[str, str, str, str] = ("lq1", "lk1", "lq2", "lk2")
+    q_name: str = "q"
+    k_name: str = "k"
+    v_name: str = "v"
+    o_name: str = "o"
+
+
+@dataclass(frozen=True)
 class StateSpaceSpec(PartSpec):
     """A selective state-space mixer with a scalar decay a head.  W_in h = [z | x | B | C | dt] with z, x of ``n_heads`` *
     ``head_dim``, B and C of ``n_groups`` * ``state`` and dt of ``n_heads`` entries.  x, B and C pass a causal convolution
@@ -389,7 +422,10 @@ class MixtureSpec(PartSpec):
     ``scores`` "sigmoid": a score is the sigmoid of the logit; the choice reads score + ``correction_name`` (a stored vector [n_experts];
     None: the score alone), first among ``n_groups`` equal runs of neighbouring experts (a run counts the sum of its ``group_best``
     largest; only the ``keep_groups`` best runs stay), then the ``top_k`` largest of what stays; the weights are the chosen experts'
-    plain scores, not renormalised, times ``route_scale``."""
+    plain scores, not renormalised, times ``route_scale``.
+    ``scores`` "softmax_all" takes a ``correction_name`` too: the choice reads score + correction, the weights are the plain scores.
+    ``n_identity``: the router has so many more outputs behind the experts' (and the correction so many more entries); each stands for an
+    expert without tensors whose output is its input."""
     hidden: int
     n_experts: int
     top_k: int
@@ -411,6 +447,7 @@ class MixtureSpec(PartSpec):
     n_groups: int = 1
     keep_groups: int = 1
     group_best: int = 2
+    n_identity: int = 0
 
 
 # ------------------------------------------------------------------ layers and the model
@@ -421,7 +458,8 @@ class LayerSpec:
 
     ``arrangement`` names an entry of ``parts.registry.ARRANGEMENTS``; "pre_norm" is
     x += mixer(norm(x)); x += ffn(norm(x))  (pico-engine src/pico_engine/model.py:167-237); "parallel" is
-    x += mixer(norm1(x)) + ffn(norm2(x)), both halves reading the same x; "post_norm" is
+    x += mixer(norm1(x)) + ffn(norm2(x)), both halves reading the same x; "parallel_one_norm" is
+    x += mixer(h) + ffn(h) with h = norm(x), one norm (``mixer_norm``) for both; "post_norm" is
     x += scale1 * norm1(mixer(x)); x += scale2 * norm2(ffn(x)): the sublayers read the stream as it is and the norms
     act on their outputs (``mixer_scale`` / ``feed_forward_scale`` name the scale vectors; None: no scale); "sandwich" is
     x += out_norm1(mixer(norm1(x))); x += out_norm2(ffn(norm2(x))) with a norm before and one after each sublayer

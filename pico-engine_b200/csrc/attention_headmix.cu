@@ -37,6 +37,7 @@ struct HeadMixArgs {
     float* stats;                             // [tile][split][QT][H][2]
     float* opart;                             // [tile][split][QT][H][Dv]
     void* out;                                // [T][H * Dv]
+    int v_share, out_f32;                     // neighbouring key heads that read one value head (the value pool has G / v_share heads); out is float32
 };
 
 struct TileInfo { int row, t0, nq, p0; };
@@ -168,7 +169,8 @@ __global__ void __launch_bounds__(HM_THREADS) headmix_kernel(HeadMixArgs a) {
         for (int e = tid; e < G * HM_KB * Dv; e += HM_THREADS) {
             const int d = e % Dv, j = (e / Dv) % HM_KB, c = e / (Dv * HM_KB);
             float v = 0.f;
-            if (page >= 0 && kb + j < k_end) v = to_f(vp[(((size_t)page * G + c) * PE_PAGE + in_page + j) * a.v_ld + d]);
+            if (page >= 0 && kb + j < k_end)
+                v = to_f(vp[(((size_t)page * (G / a.v_share) + c / a.v_share) * PE_PAGE + in_page + j) * a.v_ld + d]);
             kv_s[((size_t)c * HM_KB + j) * pitch + d] = v;
         }
         const float* wsrc = p_s;
@@ -211,7 +213,8 @@ __global__ void __launch_bounds__(HM_THREADS) headmix_kernel(HeadMixArgs a) {
         if (e < total) {
             const int d = e % Dv, i = (e / Dv) % QT, h = e / (Dv * QT);
             if (a.splits == 1) {
-                if (i < ti.nq) ((T*)a.out)[((size_t)(ti.t0 + i) * H + h) * Dv + d] = from_f<T>(acc[r]);
+                const size_t at = ((size_t)(ti.t0 + i) * H + h) * Dv + d;
+                if (i < ti.nq) { if (a.out_f32) ((float*)a.out)[at] = acc[r]; else ((T*)a.out)[at] = from_f<T>(acc[r]); }
             } else {
                 a.opart[(((size_t)blockIdx.x * a.splits + split) * QT + i) * H * Dv + (size_t)h * Dv + d] = acc[r];
             }
@@ -231,7 +234,8 @@ __global__ void headmix_reduce_kernel(HeadMixArgs a) {
         const int i = e / HD, r = e % HD;
         float s = 0.f;
         for (int sp = 0; sp < a.splits; ++sp) s += a.opart[(((size_t)blockIdx.x * a.splits + sp) * a.QT + i) * HD + r];
-        ((T*)a.out)[(size_t)(ti.t0 + i) * HD + r] = from_f<T>(s);
+        const size_t at = (size_t)(ti.t0 + i) * HD + r;
+        if (a.out_f32) ((float*)a.out)[at] = s; else ((T*)a.out)[at] = from_f<T>(s);
     }
 }
 
@@ -275,8 +279,10 @@ extern "C" int pe_attention_headmix(const void* q, int q_stride, void* out, cons
                                     const int* table, int table_stride, const int* tok_pos, const int* tok_row,
                                     const int* tiles, int n_runs, int tile_tokens, int T, int H, int G, int D, int Dv,
                                     int window, float scale, const void* sink, int sink_dtype, const void* mix, int mix_dtype,
-                                    int QT, int splits, float* scratch, const float* slopes, int keep_first, int v_ld, void* stream) {
+                                    int QT, int splits, float* scratch, const float* slopes, int keep_first, int v_ld, int v_share,
+                                    int out_f32, void* stream) {
     if (T <= 0) return 0;
+    if (v_share < 1 || G % v_share) return PE_ERR_UNSUPPORTED;
     if (v_ld <= 0) v_ld = Dv;
     if (v_ld < Dv || keep_first < 0) return PE_ERR_UNSUPPORTED;
     if (H <= 0 || G <= 0 || H % G || QT < 1 || splits < 1 || splits > 65535 || (tiles && (tile_tokens % QT || n_runs <= 0)))
@@ -287,7 +293,7 @@ extern "C" int pe_attention_headmix(const void* q, int q_stride, void* out, cons
     const int n_tiles = tiles ? n_runs * (tile_tokens / QT) : T;
     HeadMixArgs a = {q, q_stride, k_pool, v_pool, table, table_stride, tok_pos, tok_row, tiles, tile_tokens, H, G, D, Dv, window,
                      scale, sink, sink_dtype, mix, mix_dtype, QT, splits, slopes, keep_first, v_ld, scratch,
-                     scratch + (size_t)n_tiles * splits * QT * H * 2, out};
+                     scratch + (size_t)n_tiles * splits * QT * H * 2, out, v_share, out_f32};
     cudaStream_t s = (cudaStream_t)stream;
     const int nacc = (int)(((size_t)H * QT * Dv + HM_THREADS - 1) / HM_THREADS);
     if (dtype == PE_F32) {

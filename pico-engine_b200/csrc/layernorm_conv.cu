@@ -465,3 +465,104 @@ extern "C" int pe_layernorm_add(float* x, const void* y, int y_dtype, const void
     PE_LAUNCH_CHECK();
     return 0;
 }
+
+// ---------------------------------------------------------------- sums into the stream, then the next layer norm
+// x[t] += y[t] (float32 or bfloat16; null: nothing) + rw[t * rw_ld] * rows[t] (in out's dtype, or float32 / bfloat16 by rows_dtype; null:
+// nothing) on the float32 stream, and with `out` also out[t] = layernorm(x[t]) * w + b of the row as it then stands.  A block a token.
+template <typename TO, int NV>
+__global__ void __launch_bounds__(LN_THREADS) add_layernorm_vec_kernel(float* x, const void* y, int y_dtype, const void* rows, int rows_dtype,
+                                                                       const float* rw, int rw_ld, const void* w, int w_dtype, const void* b,
+                                                                       int b_dtype, float eps, int H, TO* out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const int n4 = H / 4;
+    const size_t row4 = (size_t)blockIdx.x * n4;
+    const float a = rows ? rw[(size_t)blockIdx.x * rw_ld] : 0.f;
+    float4 xv[NV];
+    float s = 0.f;
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+        const int i = threadIdx.x + LN_THREADS * v;
+        if (i < n4) {
+            xv[v] = ln_load4(x, row4 + i);
+            if (y) {
+                const float4 f = ln_load4_as_f(y, y_dtype, row4 + i);
+                xv[v].x += f.x; xv[v].y += f.y; xv[v].z += f.z; xv[v].w += f.w;
+            }
+            if (a != 0.f) {
+                const float4 f = ln_load4_as_f(rows, rows_dtype, row4 + i);
+                xv[v].x = fmaf(a, f.x, xv[v].x); xv[v].y = fmaf(a, f.y, xv[v].y); xv[v].z = fmaf(a, f.z, xv[v].z); xv[v].w = fmaf(a, f.w, xv[v].w);
+            }
+            ln_store4(x, row4 + i, xv[v]);
+            s += (xv[v].x + xv[v].y) + (xv[v].z + xv[v].w);
+        }
+    }
+    if (!out) return;
+    const float mean = block_sum(s, scratch) / (float)H;
+    float q = 0.f;
+#pragma unroll
+    for (int v = 0; v < NV; ++v)
+        if (threadIdx.x + LN_THREADS * v < n4) {
+            const float c = xv[v].x - mean, d = xv[v].y - mean, e = xv[v].z - mean, f = xv[v].w - mean;
+            q += (c * c + d * d) + (e * e + f * f);
+        }
+    const float rstd = 1.0f / sqrtf(block_sum(q, scratch) / (float)H + eps);
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+        const int i = threadIdx.x + LN_THREADS * v;
+        if (i < n4) {
+            const float4 wv = ln_load4_as_f(w, w_dtype, i), bv = ln_load4_as_f(b, b_dtype, i);
+            ln_store4(out, row4 + i, make_float4(fmaf((xv[v].x - mean) * rstd, wv.x, bv.x), fmaf((xv[v].y - mean) * rstd, wv.y, bv.y),
+                                                 fmaf((xv[v].z - mean) * rstd, wv.z, bv.z), fmaf((xv[v].w - mean) * rstd, wv.w, bv.w)));
+        }
+    }
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(LN_THREADS) add_layernorm_kernel(float* x, const void* y, int y_dtype, const void* rows, int rows_dtype,
+                                                                   const float* rw, int rw_ld, const void* w, int w_dtype, const void* b,
+                                                                   int b_dtype, float eps, int H, TO* out) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const size_t at = (size_t)blockIdx.x * H;
+    const float a = rows ? rw[(size_t)blockIdx.x * rw_ld] : 0.f;
+    float s = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) {         // (a thread rereads only entries it wrote itself)
+        float n = x[at + i];
+        if (y) n += load_as_f(y, y_dtype, at + i);
+        if (a != 0.f) n = fmaf(a, load_as_f(rows, rows_dtype, at + i), n);
+        x[at + i] = n;
+        s += n;
+    }
+    if (!out) return;
+    const float mean = block_sum(s, scratch) / (float)H;
+    float q = 0.f;
+    for (int i = threadIdx.x; i < H; i += blockDim.x) { const float d = x[at + i] - mean; q = fmaf(d, d, q); }
+    const float rstd = 1.0f / sqrtf(block_sum(q, scratch) / (float)H + eps);
+    for (int i = threadIdx.x; i < H; i += blockDim.x)
+        out[at + i] = from_f<TO>(fmaf((x[at + i] - mean) * rstd, load_as_f(w, w_dtype, i), load_as_f(b, b_dtype, i)));
+}
+
+extern "C" int pe_add_layernorm(float* x, const void* y, int y_dtype, const void* rows, int rows_dtype, const float* rw, int rw_ld,
+                                const void* w, int w_dtype, const void* b, int b_dtype, float eps, int T, int H, void* out, int out_dtype,
+                                void* stream) {
+    if (T <= 0) return 0;
+    if (H <= 0 || (out && (!w || !b)) || (rows && !rw) || (out && out_dtype != PE_BF16 && out_dtype != PE_F32)) return PE_ERR_UNSUPPORTED;
+    cudaStream_t s = (cudaStream_t)stream;
+    const bool obf = out && out_dtype == PE_BF16;
+    const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)rows | (uintptr_t)w | (uintptr_t)b | (uintptr_t)out;
+#define ALN(K, TO) PE_TRY(pe_launch(K, T, LN_THREADS, 0, s, x, y, y_dtype, rows, rows_dtype, rw, rw_ld, w, w_dtype, b, b_dtype, eps, H, (TO*)out))
+#define ALN_V(NV) do { if (obf) ALN((add_layernorm_vec_kernel<bf16, NV>), bf16); else ALN((add_layernorm_vec_kernel<float, NV>), float); } while (0)
+    if (H % 4 == 0 && H <= 4 * 4 * LN_THREADS && !(all & 15)) {
+        const int nv = (H / 4 + LN_THREADS - 1) / LN_THREADS;
+        if (nv <= 1) ALN_V(1); else if (nv == 2) ALN_V(2); else ALN_V(4);
+    } else {
+        if (obf) ALN((add_layernorm_kernel<bf16>), bf16); else ALN((add_layernorm_kernel<float>), float);
+    }
+#undef ALN_V
+#undef ALN
+    PE_LAUNCH_CHECK();
+    return 0;
+}

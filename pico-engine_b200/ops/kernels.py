@@ -726,6 +726,31 @@ def layernorm(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, eps: fl
     return out
 
 
+def add_layernorm(x: torch.Tensor, y: Optional[torch.Tensor], norm: Optional[tuple] = None, out_dtype: Optional[torch.dtype] = None,
+                  rows: Optional[torch.Tensor] = None, row_weights: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """x += y (float32 or bfloat16 rows [T, W], or None) + row_weights[t] * rows[t] (``rows`` [T, W] in either dtype, ``row_weights`` a float32
+    view [T] of any stride; None: nothing) on the float32 stream.  ``norm`` = (weight, bias, eps): also returns the layer norm of the rows
+    as they then stand, in ``out_dtype``; one kernel either way."""
+    T, W = x.shape
+    _need(x, "x", torch.float32)
+    if y is not None:
+        _need(y, "y", None, (T, W))
+    if rows is not None:
+        _need(rows, "rows", None, (T, W))
+        if row_weights is None or row_weights.dtype != torch.float32 or tuple(row_weights.shape) != (T,) or not row_weights.is_cuda:
+            raise KernelError("rows that are added need a float32 weight each")
+    out, w, b, eps = None, None, None, 0.0
+    if norm is not None:
+        w, b, eps = norm
+        _need(w, "weight", None, (W,)); _need(b, "bias", None, (W,))
+        out = torch.empty(T, W, dtype=out_dtype, device=x.device)
+    check(mixers().pe_add_layernorm(x.data_ptr(), _ptr(y), 0 if y is None else _code(y, "y"), _ptr(rows), 0 if rows is None else _code(rows, "rows"),
+                                    None if rows is None else row_weights.data_ptr(), 0 if rows is None else row_weights.stride(0), _ptr(w),
+                                    0 if w is None else _code(w, "weight"), _ptr(b), 0 if b is None else _code(b, "bias"), float(eps), T, W,
+                                    _ptr(out), 0 if out is None else _code(out, "out"), stream_ptr()), "add_layernorm")
+    return out
+
+
 def _state_args(state: torch.Tensor, offset: int, elems: int):
     """Address of element ``offset`` of slot 0 of a float32 state area [slots, elems of all parts] and its row stride."""
     _need(state, "state", torch.float32)
@@ -855,13 +880,15 @@ def attention_headmix(q: torch.Tensor, q_stride: int, n_heads: int, n_kv: int, h
                       k_pool: torch.Tensor, v_pool: torch.Tensor, block_table: torch.Tensor, table_stride: int,
                       tok_pos: torch.Tensor, tok_row: torch.Tensor, window: Optional[int], scale: float,
                       sink: Optional[torch.Tensor], mix: Optional[torch.Tensor], ctx, slopes: Optional[torch.Tensor] = None,
-                      keep_first: int = 0, values_in_keys: bool = False) -> torch.Tensor:
+                      keep_first: int = 0, values_in_keys: bool = False, v_share: int = 1, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """Attention of the step's tokens over the cache with the softmax weights mixed across heads (``mix`` [H, H]; None: not
     mixed) and a sink logit a head in the denominator (``sink`` [H]; None: none); [T, H * Dv] in q's dtype.  ``slopes``
     float32 [H]: slope_h * (i - j) is taken off the score of query i and key j.  ``keep_first``: with a window, the first so many
     keys of a sequence stay visible.  ``values_in_keys``: a position's value is the first Dv entries of its key row
-    (``v_pool`` is not read)."""
+    (``v_pool`` is not read).  ``v_share`` neighbouring key heads read one value head (``v_pool`` then has n_kv / v_share heads) and
+    ``out_dtype`` float32 keeps the outputs unrounded: both are known to the float32-FMA kernel only."""
     T = tok_pos.shape[0]
+    plain_out = v_share == 1 and out_dtype in (None, q.dtype)
     _need(q, "q"); _need(k_pool, "k_pool", q.dtype)
     if values_in_keys:
         if v_head_dim > head_dim:
@@ -870,7 +897,7 @@ def attention_headmix(q: torch.Tensor, q_stride: int, n_heads: int, n_kv: int, h
     else:
         _need(v_pool, "v_pool", q.dtype)
         v_ld = v_head_dim
-    if tuple(k_pool.shape[1:]) != (n_kv, PAGE, head_dim) or tuple(v_pool.shape[1:]) != (n_kv, PAGE, v_ld):
+    if tuple(k_pool.shape[1:]) != (n_kv, PAGE, head_dim) or tuple(v_pool.shape[1:]) != (n_kv // v_share, PAGE, v_ld):
         raise KernelError("cache pools do not have the heads and head sizes of this attention")
     if slopes is not None:
         _need(slopes, "slopes", torch.float32, (n_heads,))
@@ -880,7 +907,7 @@ def attention_headmix(q: torch.Tensor, q_stride: int, n_heads: int, n_kv: int, h
     if mix is not None:
         _need(mix, "mix", None, (n_heads, n_heads))
     sink_f32 = sink is None or sink.dtype == torch.float32
-    if (q.dtype == torch.bfloat16 and not ctx.one_token_each and sink_f32 and mix is None and not values_in_keys
+    if (plain_out and q.dtype == torch.bfloat16 and not ctx.one_token_each and sink_f32 and mix is None and not values_in_keys
             and head_dim == v_head_dim and attention_prefill_tcgen05_takes(head_dim, scale) and q_stride % 8 == 0
             and HEADMIX_TENSOR_CORES == "1"):
         # one weight a (query, key) and equal sizes of 64 or 128: the tcgen05 kernel of the plain attention, which takes the
@@ -890,7 +917,7 @@ def attention_headmix(q: torch.Tensor, q_stride: int, n_heads: int, n_kv: int, h
             tiles = ctx.scratch["prefill_tiles_128"] = prefill_tiles(ctx.lens, ctx.starts, q.device, PREFILL_TILE_TCGEN05)
         return attention_prefill_tcgen05(q, q_stride, n_heads, n_kv, head_dim, k_pool, v_pool, block_table, table_stride, tiles, T,
                                          window, scale, keep_first=keep_first, slopes=slopes, sinks=sink)
-    if (q.dtype == torch.bfloat16 and ctx.one_token_each and sink_f32 and mix is None and not values_in_keys
+    if (plain_out and q.dtype == torch.bfloat16 and ctx.one_token_each and sink_f32 and mix is None and not values_in_keys
             and head_dim == v_head_dim and attention_prefill_tcgen05_takes(head_dim, scale) and q_stride % 8 == 0
             and HEADMIX_TENSOR_CORES == "1"):
         # single tokens at the same sizes: the decode kernel of the plain attention, which knows both as well (the kernels before
@@ -905,9 +932,9 @@ def attention_headmix(q: torch.Tensor, q_stride: int, n_heads: int, n_kv: int, h
             tiles = ctx.scratch["prefill_tiles"] = prefill_tiles(ctx.lens, ctx.starts, q.device, PREFILL_TILE)
         n_runs = tiles.shape[0]
     from .workspace import scratch
-    out = torch.empty(T, n_heads * v_head_dim, dtype=q.dtype, device=q.device)
+    out = torch.empty(T, n_heads * v_head_dim, dtype=out_dtype or q.dtype, device=q.device)
     floats = all(t is None or t.dtype == torch.float32 for t in (sink, mix))
-    if q.dtype == torch.bfloat16 and HEADMIX_TENSOR_CORES == "1" and floats:
+    if plain_out and q.dtype == torch.bfloat16 and HEADMIX_TENSOR_CORES == "1" and floats:
         cg = lib.pe_attention_flashmix_group(n_heads, n_kv, head_dim, v_head_dim)
         if cg and q_stride % 2 == 0 and v_ld % 8 == 0:
             # one pass over the keys with an output for every (head, value head), then merge + sink + mixing
@@ -927,7 +954,7 @@ def attention_headmix(q: torch.Tensor, q_stride: int, n_heads: int, n_kv: int, h
                                             _ptr(mix), splits, ws.data_ptr(), _ptr(slopes), keep_first, v_ld, stream_ptr()),
                   "attention_flashmix", 2)
             return out
-    if q.dtype == torch.bfloat16 and HEADMIX_TENSOR_CORES in ("1", "two-pass") and floats and plain_mask:
+    if plain_out and q.dtype == torch.bfloat16 and HEADMIX_TENSOR_CORES in ("1", "two-pass") and floats and plain_mask:
         kb = headmix_mma_key_block(n_heads, n_kv, head_dim, v_head_dim)
         if kb:
             # bfloat16: the tensor-core kernel; tiles of 16 tokens, ranges of at least two key blocks
@@ -955,7 +982,7 @@ def attention_headmix(q: torch.Tensor, q_stride: int, n_heads: int, n_kv: int, h
                                    n_runs, PREFILL_TILE, T, n_heads, n_kv, head_dim, v_head_dim, window or 0, float(scale),
                                    _ptr(sink), 0 if sink is None else _code(sink, "sink"), _ptr(mix),
                                    0 if mix is None else _code(mix, "mix"), qt, splits, ws.data_ptr(), _ptr(slopes), keep_first, v_ld,
-                                   stream_ptr()),
+                                   v_share, 1 if out.dtype == torch.float32 and q.dtype != torch.float32 else 0, stream_ptr()),
           "attention_headmix", 2 + (splits > 1))
     return out
 
@@ -1578,3 +1605,101 @@ def stream_mix(src: torch.Tensor, n_streams: int, dst: Optional[torch.Tensor] = 
                                 _ptr(norm_weight), 0 if norm_weight is None else _code(norm_weight, "norm_weight"), float(eps), _ptr(h),
                                 0 if h is None else _code(h, "h"), T, S, W, stream_ptr()), "stream_mix")
     return h
+
+
+# ---------------------------------------------------------------------------- heads with two maps; sublayers that share their products
+
+def heads_norm_store(proj: torch.Tensor, n_heads: int, n_kv: int, v_heads: int, head_dim: int, v_head_dim: int, q_weight: Optional[torch.Tensor],
+                     k_weight: Optional[torch.Tensor], eps: float, freq: Optional[torch.Tensor], rot_dims: int, tok_pos: torch.Tensor,
+                     tok_row: torch.Tensor, k_pool: Optional[torch.Tensor], v_pool: Optional[torch.Tensor], block_table: Optional[torch.Tensor],
+                     table_stride: int) -> None:
+    """On rows proj [T, ld] that begin with n_heads query, n_kv key rows of ``head_dim`` and ``v_heads`` value rows of ``v_head_dim`` entries:
+    every query and key row RMS-normed over its entries (``q_weight`` / ``k_weight`` [head_dim] shared by all of them; None: not normed),
+    entries i and i + rot_dims / 2 turned by pos * freq[i]; queries are rewritten in place, keys and values go to their cache pages
+    (``k_pool`` None: they do not)."""
+    from .library import joined
+    T, ld = proj.shape
+    _need(proj, "proj"); _need(tok_pos, "tok_pos", torch.int32, (T,)); _need(tok_row, "tok_row", torch.int32, (T,))
+    for w, name in ((q_weight, "q_weight"), (k_weight, "k_weight")):
+        if w is not None:
+            _need(w, name, None, (head_dim,))
+    if rot_dims:
+        _need(freq, "freq", torch.float32, (rot_dims // 2,))
+    store = k_pool is not None
+    if store:
+        _need(k_pool, "k_pool", proj.dtype); _need(v_pool, "v_pool", proj.dtype); _need(block_table, "block_table", torch.int32)
+        if tuple(k_pool.shape[1:]) != (n_kv, PAGE, head_dim) or tuple(v_pool.shape[1:]) != (v_heads, PAGE, v_head_dim):
+            raise KernelError(f"cache pools must be [pages, {n_kv}, {PAGE}, {head_dim}] and [pages, {v_heads}, {PAGE}, {v_head_dim}], "
+                              f"not {tuple(k_pool.shape)} and {tuple(v_pool.shape)}")
+    check(joined().pe_heads_norm_store(proj.data_ptr(), _code(proj, "proj"), ld, T, n_heads, n_kv, v_heads, head_dim, v_head_dim, _ptr(q_weight),
+                                       0 if q_weight is None else _code(q_weight, "q_weight"), _ptr(k_weight),
+                                       0 if k_weight is None else _code(k_weight, "k_weight"), float(eps), _ptr(freq), rot_dims, tok_pos.data_ptr(),
+                                       tok_row.data_ptr(), _ptr(k_pool), _ptr(v_pool), _ptr(block_table), table_stride, 1 if store else 0,
+                                       stream_ptr()), "heads_norm_store")
+
+
+def map_difference(maps: torch.Tensor, n_heads: int, n_kv: int, v_head_dim: int, lam: float, eps: float, scale: float, out: torch.Tensor,
+                   out_col: int) -> None:
+    """Columns ``out_col`` .. of out [T, ld] from the maps' float32 outputs [T, n_kv * 2 * (n_heads / n_kv) * Dv], laid out key/value head by
+    key/value head as [map 1 of its heads | map 2 of its heads]: (a1 - lam a2) / sqrt(mean((a1 - lam a2)^2) + eps) * scale a head."""
+    from .library import joined
+    T = maps.shape[0]
+    _need(maps, "maps", torch.float32, (T, 2 * n_heads * v_head_dim)); _need(out, "out")
+    if out.shape[0] != T:
+        raise KernelError("out needs a row a token")
+    check(joined().pe_map_difference(maps.data_ptr(), T, n_heads, n_kv, v_head_dim, float(lam), float(eps), float(scale), out.data_ptr(),
+                                     _code(out, "out"), out.shape[1], out_col, stream_ptr()), "map_difference")
+
+
+def attention_maps(q: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, v_head_dim: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
+                   block_table: torch.Tensor, table_stride: int, tok_pos: torch.Tensor, tok_row: torch.Tensor, window: Optional[int], scale: float,
+                   lam: float, eps: float, out_scale: float, out: torch.Tensor, out_col: int, ctx) -> None:
+    """Differential attention of the step's tokens over the cache into columns ``out_col`` .. of out [T, ld] (a head = ``v_head_dim`` columns,
+    heads in their order).  The rows of ``q`` [T, ld2] begin with the queries laid out key/value head by key/value head as [map 1 of its
+    heads | map 2 of its heads]; ``k_pool`` has 2 n_kv heads (key/value head g's maps at 2g and 2g + 1), ``v_pool`` n_kv."""
+    maps = attention_headmix(q, q.shape[1], 2 * n_heads, 2 * n_kv, head_dim, v_head_dim, k_pool, v_pool, block_table, table_stride, tok_pos, tok_row,
+                             window, scale, None, None, ctx, v_share=2, out_dtype=torch.float32)
+    map_difference(maps, n_heads, n_kv, v_head_dim, lam, eps, out_scale, out, out_col)
+
+
+def side_act(src: torch.Tensor, gate_col: int, up_col: int, n: int, activation: str, out: torch.Tensor, out_col: int,
+             col_weights: Optional[torch.Tensor] = None, group: int = 0, n_groups: int = 0) -> None:
+    """out[t, out_col + c] = act(src[t, gate_col + c]) * src[t, up_col + c] for c < n (``up_col`` < 0: act alone), formed in float32;
+    ``col_weights`` float32 [T, >= n_groups]: column c is also multiplied by col_weights[t, min(c // group, n_groups - 1)] (a zero weight
+    gives an exact zero)."""
+    from .library import joined
+    T, ld = src.shape
+    _need(src, "src"); _need(out, "out", src.dtype)
+    if out.shape[0] != T:
+        raise KernelError("out needs a row a token")
+    if col_weights is not None:
+        _need(col_weights, "col_weights", torch.float32)
+        if col_weights.shape[0] != T or col_weights.shape[1] < n_groups:
+            raise KernelError("col_weights needs a row a token and a column a group")
+    check(joined().pe_side_act(src.data_ptr(), _code(src, "src"), ld, gate_col, up_col, T, n, GATE_ACTIVATIONS[activation], _ptr(col_weights),
+                               0 if col_weights is None else col_weights.shape[1], group, n_groups, out.data_ptr(), out.shape[1], out_col,
+                               stream_ptr()), "side_act")
+
+
+ROUTE_ROWS_MAX = 1024      # RR_MAX_N of csrc/joined_ops.cu
+
+
+def route_rows(h: torch.Tensor, router: torch.Tensor, n_outputs: int, n_experts: int, top_k: int, correction: Optional[torch.Tensor], gate: bool,
+               factor: float = 1.0, ids: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Routing weights float32 [T, n_experts + gate + (n_outputs > n_experts)] of rows h [T, K] that are normed already.  Scores are the
+    softmax over the first ``n_outputs`` products with ``router`` [n_outputs + gate, K] (h's dtype, float32 sums); the ``top_k`` largest of
+    score + correction are chosen and weighted by factor * score.  Columns: experts 0 .. n_experts - 1 (zero where not chosen); with
+    ``gate`` the sigmoid of the last row's product; where the router has more outputs than experts, the sum of the weights of the chosen
+    ones among those.  ``ids`` int32 [T, top_k] receives the chosen."""
+    from .library import joined
+    T, K = h.shape
+    _need(h, "h"); _need(router, "router", h.dtype, (n_outputs + (1 if gate else 0), K))
+    if correction is not None:
+        _need(correction, "correction", None, (n_outputs,))
+    if ids is not None:
+        _need(ids, "ids", torch.int32, (T, top_k))
+    out = torch.empty(T, n_experts + (1 if gate else 0) + (1 if n_outputs > n_experts else 0), dtype=torch.float32, device=h.device)
+    check(joined().pe_route_rows(h.data_ptr(), _code(h, "h"), router.data_ptr(), K, n_outputs, n_experts, 1 if gate else 0, _ptr(correction),
+                                 0 if correction is None else _code(correction, "correction"), top_k, float(factor), out.data_ptr(), _ptr(ids), T,
+                                 stream_ptr()), "route_rows")
+    return out

@@ -28,6 +28,9 @@ GATED_SOURCES = ("linear_attention.cu", "linear_attention_tiles.cu", "gated_ops.
 # The kernels of the state-space mixer (short convolution with silu, the recurrence with a scalar decay, gate then norm) and of
 # attention over one low-rank row per position.
 STATE_SOURCES = ("state_space.cu", "latent_ops.cu")
+# The kernels of sublayers that read the same rows and share their first and last product, of heads with several maps, and of routers
+# that read normed rows.
+JOINED_SOURCES = ("joined_ops.cu",)
 HEAD_DIM_SOURCES = ("attention_decode.cu", "attention_prefill.cu", "attention_prefill_tcgen05.cu")      # compiled per head size
 
 _SIGNATURES = {
@@ -59,11 +62,12 @@ _SIGNATURES = {
 _MIXER_SIGNATURES = {
     "pe_layernorm": [P, P, P, I, P, I, F, P, I, I, I, P],
     "pe_layernorm_add": [P, P, I, P, I, P, I, F, I, I, P, I, P, I, F, P, I, P],
+    "pe_add_layernorm": [P, P, I, P, I, P, I, P, I, P, I, F, I, I, P, I, P],
     "pe_causal_conv_add": [P, P, I, P, LL, P, P, P, P, I, I, I, I, P],
     "pe_conv_state_update": [P, P, LL, P, P, P, I, I, I, P],
     "pe_dual_layernorm_conv": [P, P, I, P, I, P, I, P, P, P, I, P, I, P, I, P, P, I, LL, P, P, P, P, F, I, I, I, I, I, P],
     "pe_mingru": [P, I, P, LL, P, P, P, P, P, I, I, I, I, P, P],
-    "pe_attention_headmix": [P, I, P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, I, I, I, P, P, I, I, P],
+    "pe_attention_headmix": [P, I, P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, I, I, I, P, P, I, I, I, I, P],
     "pe_qknorm_store": [P, I, I, I, I, I, I, P, I, P, I, F, P, P, P, P, P, I, I, P],
     "pe_attention_flashmix": [P, I, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, P, P, I, P, P, I, I, P],
     "pe_attention_headmix_mma": [P, I, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, P, I, P, P],
@@ -95,6 +99,13 @@ _STATE_SIGNATURES = {
     "pe_latent_prepare": [P, I, I, I, I, I, I, I, I, P, I, F, P, I, P, P, P, P, P, P, I, I, I, P, I, P],
     "pe_rmsnorm_cols": [P, I, I, I, I, P, I, F, P, I, P],
     "pe_head_gate": [P, I, P, I, I, I, I, I, P, P],
+}
+
+_JOINED_SIGNATURES = {
+    "pe_heads_norm_store": [P, I, I, I, I, I, I, I, I, P, I, P, I, F, P, I, P, P, P, P, P, I, I, P],
+    "pe_map_difference": [P, I, I, I, I, F, F, F, P, I, I, I, P],
+    "pe_side_act": [P, I, I, I, I, I, I, I, P, I, I, I, P, I, I, P],
+    "pe_route_rows": [P, I, P, I, I, I, I, P, I, I, F, P, P, I, P],
 }
 
 _EXTRA_SIGNATURES = {
@@ -212,6 +223,21 @@ def state_space() -> ctypes.CDLL:
         lib.pe_state_space_scratch_floats.restype = c_longlong
         _state = lib
     return _state
+
+
+_joined = None
+
+
+def joined() -> ctypes.CDLL:
+    """The library of the kernels of sublayers that share their first and last product, of heads with several maps and of routers that
+    read normed rows; compiled at the first call."""
+    global _joined
+    if _joined is None:
+        lib = build.load("joined", JOINED_SOURCES)
+        declare(lib, _JOINED_SIGNATURES)
+        lib.pe_set_pdl(0 if os.environ.get("PICO_ENGINE_PDL", "1") == "0" else 1)
+        _joined = lib
+    return _joined
 
 
 _extras = None

@@ -17,7 +17,9 @@ from .mixture import Mixture
 from .attention_latent import LatentAttention
 from .state_space import StateSpace
 from .streams import StreamMix
-from .block import Layer, parallel, post_norm, pre_norm, sandwich, streams
+from .attention_differential import DifferentialAttention
+from .joined import JoinedSublayers
+from .block import Layer, parallel, parallel_one_norm, post_norm, pre_norm, sandwich, streams
 from .model import DecoderModel
 
 __all__ = ["ARRANGEMENTS", "FEED_FORWARDS", "MIXERS", "NORMS", "POSITIONS", "FeedForward", "KVView", "Mixer", "Norm",
@@ -25,4 +27,5 @@ __all__ = ["ARRANGEMENTS", "FEED_FORWARDS", "MIXERS", "NORMS", "POSITIONS", "Fee
            "register_mixer", "register_norm", "register_position", "RMSNorm", "NoPosition", "RotaryHalf",
            "GQAAttention", "SwiGLU", "Layer", "pre_norm", "DecoderModel", "LayerNorm", "SinusoidAdd", "CausalConvAdd",
            "HeadMixAttention", "MinGRU", "DenseMLP", "parallel", "GatedMLP", "LinearAttention", "GatedAttention", "BranchSum", "Mixture",
-           "LatentAttention", "StateSpace", "post_norm", "sandwich", "StreamMix", "streams"]
+           "LatentAttention", "StateSpace", "post_norm", "sandwich", "StreamMix", "streams", "DifferentialAttention",
+           "JoinedSublayers", "parallel_one_norm"]

@@ -24,6 +24,14 @@ def halves_frequencies(spec: RotaryHalvesSpec, device):
     half = spec.dims // 2
     f = [spec.base ** (-2.0 * i / spec.dims) for i in range(half)]
     magnitude = 1.0
+    if spec.bands is not None:
+        if spec.stretch is not None:
+            raise ConfigError("a rotation is stretched either by a ramp over its entries or by its wavelengths")
+        factor, low, high, original = spec.bands
+        for i in range(half):
+            turns = original * f[i] / (2.0 * math.pi)      # how often the entry turns within the original context
+            s = min(max((turns - low) / (high - low), 0.0), 1.0)
+            f[i] = (1.0 - s) * f[i] / factor + s * f[i]
     if spec.stretch is not None and half:
         factor, original, fast, slow = spec.stretch
 

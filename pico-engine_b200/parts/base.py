@@ -83,6 +83,7 @@ class StepContext:
     pending: Optional[torch.Tensor] = None  # a product [T, hidden] that still has to be added to the residual stream
     pending_norm: Optional["Norm"] = None   # the norm that product passes on its way into the stream (None: it is added as it is)
     pending_streams: Optional["Part"] = None  # how it enters a residual of several streams (a StreamMix)
+    pending_rows: Optional[tuple] = None    # (rows [T, hidden], weights [T]): rows times a number a token that are added with the pending product
     stream_source: Optional[torch.Tensor] = None  # the one matrix [T, hidden] that all streams still equal, before the first sum into them
 
     # A part whose product comes out of the library may leave the sum into the residual stream pending, so
@@ -90,9 +91,10 @@ class StepContext:
     # that declare ``takes_pending`` through ``normed``, everyone else through the arrangement.  A sublayer's
     # output that is normed before it is added (``defer_normed_add``) waits the same way: that norm, the sum and
     # the next reader's norm are then one pass over the rows.
-    def defer_add(self, x: torch.Tensor, y: torch.Tensor) -> None:
+    def defer_add(self, x: torch.Tensor, y: torch.Tensor, rows: Optional[tuple] = None) -> None:
+        """x += y, left pending; ``rows`` = (r [T, hidden], w float32 [T]): x += y + w[t] * r[t]."""
         self.settle(x)
-        self.pending = y
+        self.pending, self.pending_rows = y, rows
 
     def defer_normed_add(self, x: torch.Tensor, y: torch.Tensor, norm: "Norm") -> None:
         """x += norm(y), left pending."""
@@ -105,9 +107,11 @@ class StepContext:
             if self.pending_streams is not None:
                 self._mix_streams(x, dst=x)
                 return
-            y, n = self.pending, self.pending_norm
-            self.pending = self.pending_norm = None
-            if n is None:
+            y, n, rows = self.pending, self.pending_norm, self.pending_rows
+            self.pending = self.pending_norm = self.pending_rows = None
+            if rows is not None:
+                kernels.add_layernorm(x, y.contiguous(), rows=rows[0], row_weights=rows[1])
+            elif n is None:
                 kernels.residual_add(x, y.contiguous())
             else:
                 n.add_into(x, y.contiguous())
@@ -116,8 +120,10 @@ class StepContext:
         """norm(x) in the step's dtype, after what is pending has been added to x."""
         if self.pending is None:
             return norm.forward(x, self.dtype)
-        y, n = self.pending, self.pending_norm
-        self.pending = self.pending_norm = None
+        y, n, rows = self.pending, self.pending_norm, self.pending_rows
+        self.pending = self.pending_norm = self.pending_rows = None
+        if rows is not None:
+            return norm.add_forward(x, y.contiguous(), self.dtype, rows)
         if n is None:
             return norm.add_forward(x, y.contiguous(), self.dtype)
         return n.add_into(x, y.contiguous(), then=norm, out_dtype=self.dtype)
@@ -211,10 +217,13 @@ class Norm(Part):
     def forward(self, x: torch.Tensor, out_dtype: torch.dtype, rows_index: Optional[torch.Tensor] = None) -> torch.Tensor:
         raise NotImplementedError
 
-    def add_forward(self, x: torch.Tensor, y: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
-        """x += y in place, then forward(x); norms override this to do both in one pass."""
+    def add_forward(self, x: torch.Tensor, y: torch.Tensor, out_dtype: torch.dtype, rows: Optional[tuple] = None) -> torch.Tensor:
+        """x += y in place (``rows`` = (r, w): and w[t] * r[t]), then forward(x); norms override this to do both in one pass."""
         from ..ops import kernels
-        kernels.residual_add(x, y)
+        if rows is not None:
+            kernels.add_layernorm(x, y, rows=rows[0], row_weights=rows[1])
+        else:
+            kernels.residual_add(x, y)
         return self.forward(x, out_dtype)
 
     def add_into(self, x: torch.Tensor, y: torch.Tensor, then: Optional["Norm"] = None, out_dtype: Optional[torch.dtype] = None):
@@ -270,6 +279,25 @@ class SharedProducts:
 
     def gate_job(self, rows, col: int, scale: float):
         """kernels.GatedRows: norm, gate and the weight of this mixer."""
+        raise NotImplementedError
+
+
+class JoinedProducts:
+    """What a sublayer (mixer or feed-forward) offers so that it can stand beside another one that reads the same normed rows: the
+    sublayers' first products are then one and so are their last products, whose sum over columns adds the sublayers up
+    (``parts/joined.py``).  Between the two a sublayer reads its columns of the first product's rows and writes its columns of the rows
+    of the last one."""
+
+    def can_join(self) -> bool:
+        return False
+
+    def lend_products(self):
+        """(first weight [rows, hidden], last weight [hidden, columns]); the sublayer keeps neither after this."""
+        raise NotImplementedError
+
+    def fill_side(self, proj, col: int, side, side_col: int, h, ctx, cache_entry: Optional[int] = None, owns_cache: bool = True):
+        """Columns ``side_col`` .. of ``side`` from columns ``col`` .. of ``proj`` (and the normed rows h).  Returns None, or (rows, weights): rows
+        [T, hidden] that the sublayer's output also contains, times a float32 number a token."""
         raise NotImplementedError
 
 

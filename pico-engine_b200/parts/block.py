@@ -6,6 +6,7 @@ from ..config.specs import ConfigError, LayerSpec
 from .streams import StreamMix
 from ..cache import CacheNeeds
 from ..weights.loader import ParamSpec
+from .joined import JoinedSublayers
 from .base import ARRANGEMENTS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, Norm, Part, build_part, register_arrangement
 
 
@@ -77,6 +78,12 @@ class Layer:
         if spec.arrangement == "streams" and ((self.mixer is None) != (self.mixer_streams is None)
                                               or (self.feed_forward is None) != (self.feed_forward_streams is None)):
             raise ConfigError("the streams arrangement takes a stream mix for every sublayer there is")
+        self.joined = None
+        if spec.arrangement == "parallel_one_norm":
+            if spec.feed_forward_norm is not None or spec.mixer_input is not None or spec.feed_forward_input is not None:
+                raise ConfigError("the parallel_one_norm arrangement has one norm (mixer_norm) and no input filters")
+            if self.mixer is not None and self.feed_forward is not None:
+                self.joined = JoinedSublayers((self.mixer, self.feed_forward), dtype, self.mixer.device)
         if (self.mixer_input is not None and self.mixer is None) or (self.feed_forward_input is not None and self.feed_forward is None):
             raise ConfigError("an input filter needs the sublayer whose input it filters")
         try:
@@ -88,7 +95,7 @@ class Layer:
         """The parts that are there (a stand-in for an absent norm has no tensors and is left out)."""
         return tuple(p for p in (self.mixer, self.mixer_norm, self.mixer_input, self.feed_forward, self.feed_forward_norm,
                                  self.feed_forward_input, self.mixer_scale, self.feed_forward_scale, self.mixer_out_norm,
-                                 self.feed_forward_out_norm, self.mixer_streams, self.feed_forward_streams)
+                                 self.feed_forward_out_norm, self.mixer_streams, self.feed_forward_streams, self.joined)
                      if p is not None and not isinstance(p, PassThrough))
 
     def cache_needs(self):
@@ -182,6 +189,21 @@ def parallel(layer: Layer, x, ctx, entry, cache_entry, owns_cache) -> None:
             part.add_output_to(x, h, ctx)
         else:
             kernels.residual_add(x, part.apply(h, ctx).contiguous())
+
+
+@register_arrangement("parallel_one_norm")
+def parallel_one_norm(layer: Layer, x, ctx, entry, cache_entry, owns_cache) -> None:
+    """h = norm(x); x += mixer(h) + feed_forward(h): one norm whose rows both sublayers read.  Where both can, they run on one first and
+    one last product (``parts/joined.py``), whose float32 sums stay pending until the next reader's norm; else one after the other."""
+    h = ctx.normed(x, layer.mixer_norm)
+    if layer.joined is not None and layer.joined.active:
+        y, rows = layer.joined.apply(h, ctx, cache_entry, owns_cache)
+        ctx.defer_add(x, y, rows)
+        return
+    for part, where in ((layer.mixer, (entry, cache_entry, owns_cache)), (layer.feed_forward, ())):
+        if part is not None:
+            wide = {"out_dtype": x.dtype} if getattr(part, "takes_out_dtype", False) else {}
+            ctx.defer_add(x, part.apply(h, ctx, *where, **wide))
 
 
 @register_arrangement("post_norm")

@@ -6,7 +6,7 @@ import torch
 from ..config.specs import ConfigError, DenseMLPSpec, GatedMLPSpec, SwiGLUSpec
 from ..ops import kernels, linear
 from ..weights.loader import ParamSpec
-from .base import FeedForward, first_product, last_product_into, normed_rows, register_feed_forward
+from .base import FeedForward, JoinedProducts, first_product, last_product_into, normed_rows, register_feed_forward
 
 
 @register_feed_forward(SwiGLUSpec)
@@ -53,8 +53,10 @@ class SwiGLU(FeedForward):
 
 
 @register_feed_forward(DenseMLPSpec)
-class DenseMLP(FeedForward):
+class DenseMLP(FeedForward, JoinedProducts):
     """down(act(up(h))) without biases; act is the square of relu, gelu (tanh formula) or silu, computed in float32."""
+
+    takes_out_dtype = True      # apply(..., out_dtype=) gives the product's float32 sums where the caller goes on in float32
 
     def __init__(self, spec: DenseMLPSpec, dtype, device):
         super().__init__(spec, dtype, device)
@@ -75,16 +77,28 @@ class DenseMLP(FeedForward):
         up = linear(h, self.w_up, out_dtype=ctx.dtype)
         return kernels.activation(up, self.spec.activation, out=up)
 
-    def apply(self, h, ctx):
-        return linear(self._activation(h, ctx), self.w_down, out_dtype=ctx.dtype)
+    def apply(self, h, ctx, out_dtype=None):
+        return linear(self._activation(h, ctx), self.w_down, out_dtype=out_dtype or ctx.dtype)
 
     def add_output_to(self, x, h, ctx) -> None:
         """x += feed_forward(h) for rows h that are normed (and filtered) already."""
         linear(self._activation(h, ctx), self.w_down, accumulate_into=x)
 
+    # ---------------------------------------------------------------- beside another sublayer on the same rows
+    def can_join(self):
+        return True
+
+    def lend_products(self):
+        w = self.w_up, self.w_down
+        self.w_up = self.w_down = None
+        return w
+
+    def fill_side(self, proj, col, side, side_col, h, ctx, cache_entry=None, owns_cache=True):
+        kernels.side_act(proj, col, -1, self.spec.intermediate, self.spec.activation, side, side_col)
+
 
 @register_feed_forward(GatedMLPSpec)
-class GatedMLP(FeedForward):
+class GatedMLP(FeedForward, JoinedProducts):
     """down(act(gate(h)) * up(h)) without biases, gate and up as one product on concatenated weights; act is gelu
     (tanh formula), silu or relu, or the clamped form min(gate, l) sigmoid(a min(gate, l)) (clamp(up, -l, l) + 1); formed in float32."""
 
@@ -126,3 +140,16 @@ class GatedMLP(FeedForward):
         """x += scale * feed_forward(norm(x)), the norm in the first product and the sum in the last where they take the sizes."""
         last_product_into(x, self._activation(None, ctx, (x, norm)), self.w_down, scale, ctx)
         return True
+
+    # ---------------------------------------------------------------- beside another sublayer on the same rows
+    def can_join(self):
+        return self.spec.activation != "clamped_sigmoid"
+
+    def lend_products(self):
+        w = self.w_gate_up, self.w_down
+        self.w_gate_up = self.w_down = None
+        return w
+
+    def fill_side(self, proj, col, side, side_col, h, ctx, cache_entry=None, owns_cache=True):
+        n = self.spec.intermediate
+        kernels.side_act(proj, col, col + n, n, self.spec.activation, side, side_col)

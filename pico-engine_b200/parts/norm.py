@@ -29,7 +29,9 @@ class RMSNorm(Norm):
     def forward(self, x, out_dtype, rows_index=None):
         return kernels.rmsnorm(x, self.weight, self.eps, out_dtype, rows_index)
 
-    def add_forward(self, x, y, out_dtype):
+    def add_forward(self, x, y, out_dtype, rows=None):
+        if rows is not None:
+            return super().add_forward(x, y, out_dtype, rows)
         return kernels.add_rmsnorm(x, y, self.weight, self.eps, out_dtype)
 
 
@@ -55,6 +57,9 @@ class LayerNorm(Norm):
 
     def forward(self, x, out_dtype, rows_index=None):
         return kernels.layernorm(x, self.weight, self.bias, self.eps, out_dtype, rows_index)
+
+    def add_forward(self, x, y, out_dtype, rows=None):
+        return kernels.add_layernorm(x, y, (self.weight, self.bias, self.eps), out_dtype, *(rows or (None, None)))
 
     def add_into(self, x, y, then=None, out_dtype=None):
         """x += layernorm(y); with a layer norm ``then`` its rows of the new x come out of the same kernel."""
