@@ -37,6 +37,8 @@ struct HeadMixArgs {
     float* stats;                             // [tile][split][QT][H][2]
     float* opart;                             // [tile][split][QT][H][Dv]
     void* out;                                // [T][H * Dv]
+    int Hp, Gp;                               // heads of a row and of the key pool; gridDim.z blocks take H = Hp / gridDim.z and G = Gp / gridDim.z of
+                                              // them each (without mixing; more than one where all of them do not fit a block)
     int v_share, out_f32;                     // neighbouring key heads that read one value head (the value pool has G / v_share heads); out is float32
 };
 
@@ -62,6 +64,8 @@ __global__ void __launch_bounds__(HM_THREADS) headmix_kernel(HeadMixArgs a) {
     pdl_wait();
     extern __shared__ float smem[];
     const int H = a.H, G = a.G, D = a.D, Dv = a.Dv, QT = a.QT, per_kv = H / G;
+    const int h0 = blockIdx.z * H, g0 = blockIdx.z * G;
+    const size_t tile_at = (size_t)blockIdx.z * gridDim.x + blockIdx.x;
     const int pitch = max(D, Dv) + 1;
     float* q_s = smem;                                   // [QT][H][D]
     float* kv_s = q_s + (size_t)QT * H * D;              // [G][KB][pitch]
@@ -90,7 +94,7 @@ __global__ void __launch_bounds__(HM_THREADS) headmix_kernel(HeadMixArgs a) {
 
     for (int e = tid; e < QT * H * D; e += HM_THREADS) {
         const int i = e / (H * D), r = e % (H * D);
-        q_s[e] = i < ti.nq ? to_f(qg[(size_t)(ti.t0 + i) * a.q_stride + r]) : 0.f;
+        q_s[e] = i < ti.nq ? to_f(qg[(size_t)(ti.t0 + i) * a.q_stride + (size_t)h0 * D + r]) : 0.f;
     }
     if (PASS == 0) {
         for (int e = tid; e < QT * H; e += HM_THREADS) { m_s[e] = -INFINITY; l_s[e] = 0.f; }
@@ -98,10 +102,10 @@ __global__ void __launch_bounds__(HM_THREADS) headmix_kernel(HeadMixArgs a) {
         // the final maximum and denominator of every (query, head) from the ranges' partial results
         for (int e = tid; e < QT * H; e += HM_THREADS) {
             const int h = e % H;
-            const float* st = a.stats + ((size_t)blockIdx.x * a.splits * QT * H + e) * 2;
-            float M = a.sink ? load_as_f(a.sink, a.sink_dtype, h) : -INFINITY;
+            const float* st = a.stats + (tile_at * a.splits * QT * H + e) * 2;
+            float M = a.sink ? load_as_f(a.sink, a.sink_dtype, h0 + h) : -INFINITY;
             for (int s = 0; s < a.splits; ++s) M = fmaxf(M, st[(size_t)s * QT * H * 2]);
-            float den = a.sink ? expf(load_as_f(a.sink, a.sink_dtype, h) - M) : 0.f;
+            float den = a.sink ? expf(load_as_f(a.sink, a.sink_dtype, h0 + h) - M) : 0.f;
             for (int s = 0; s < a.splits; ++s) {
                 const float ms = st[(size_t)s * QT * H * 2], ls = st[(size_t)s * QT * H * 2 + 1];
                 if (ms > -INFINITY) den += ls * expf(ms - M);
@@ -124,7 +128,7 @@ __global__ void __launch_bounds__(HM_THREADS) headmix_kernel(HeadMixArgs a) {
         for (int e = tid; e < G * HM_KB * D; e += HM_THREADS) {
             const int d = e % D, j = (e / D) % HM_KB, c = e / (D * HM_KB);
             float v = 0.f;
-            if (page >= 0 && kb + j < k_end) v = to_f(kp[(((size_t)page * G + c) * PE_PAGE + in_page + j) * D + d]);
+            if (page >= 0 && kb + j < k_end) v = to_f(kp[(((size_t)page * a.Gp + g0 + c) * PE_PAGE + in_page + j) * D + d]);
             kv_s[((size_t)c * HM_KB + j) * pitch + d] = v;
         }
         __syncthreads();
@@ -141,7 +145,7 @@ __global__ void __launch_bounds__(HM_THREADS) headmix_kernel(HeadMixArgs a) {
                 float dot = 0.f;
                 for (int d = 0; d < D; ++d) dot = fmaf(qv[d], kv[d], dot);
                 s = dot * a.scale;
-                if (a.slopes) s -= a.slopes[h] * (float)(qpos - key);
+                if (a.slopes) s -= a.slopes[h0 + h] * (float)(qpos - key);
             }
             if (PASS == 0) p_s[e] = s;
             else p_s[e] = seen ? expf(s - m_s[i * H + h]) * l_s[i * H + h] : 0.f;
@@ -170,7 +174,7 @@ __global__ void __launch_bounds__(HM_THREADS) headmix_kernel(HeadMixArgs a) {
             const int d = e % Dv, j = (e / Dv) % HM_KB, c = e / (Dv * HM_KB);
             float v = 0.f;
             if (page >= 0 && kb + j < k_end)
-                v = to_f(vp[(((size_t)page * (G / a.v_share) + c / a.v_share) * PE_PAGE + in_page + j) * a.v_ld + d]);
+                v = to_f(vp[(((size_t)page * (a.Gp / a.v_share) + (g0 + c) / a.v_share) * PE_PAGE + in_page + j) * a.v_ld + d]);
             kv_s[((size_t)c * HM_KB + j) * pitch + d] = v;
         }
         const float* wsrc = p_s;
@@ -202,7 +206,7 @@ __global__ void __launch_bounds__(HM_THREADS) headmix_kernel(HeadMixArgs a) {
     }
 
     if (PASS == 0) {
-        float* st = a.stats + (((size_t)blockIdx.x * a.splits + split) * QT * H) * 2;
+        float* st = a.stats + ((tile_at * a.splits + split) * QT * H) * 2;
         for (int e = tid; e < QT * H; e += HM_THREADS) { st[2 * e] = m_s[e]; st[2 * e + 1] = l_s[e]; }
         return;
     }
@@ -213,10 +217,10 @@ __global__ void __launch_bounds__(HM_THREADS) headmix_kernel(HeadMixArgs a) {
         if (e < total) {
             const int d = e % Dv, i = (e / Dv) % QT, h = e / (Dv * QT);
             if (a.splits == 1) {
-                const size_t at = ((size_t)(ti.t0 + i) * H + h) * Dv + d;
+                const size_t at = ((size_t)(ti.t0 + i) * a.Hp + h0 + h) * Dv + d;
                 if (i < ti.nq) { if (a.out_f32) ((float*)a.out)[at] = acc[r]; else ((T*)a.out)[at] = from_f<T>(acc[r]); }
             } else {
-                a.opart[(((size_t)blockIdx.x * a.splits + split) * QT + i) * H * Dv + (size_t)h * Dv + d] = acc[r];
+                a.opart[((tile_at * a.splits + split) * QT + i) * H * Dv + (size_t)h * Dv + d] = acc[r];
             }
         }
     }
@@ -230,11 +234,12 @@ __global__ void headmix_reduce_kernel(HeadMixArgs a) {
     TileInfo ti;
     if (!hm_tile(a, blockIdx.x, ti)) return;
     const int HD = a.H * a.Dv;
+    const size_t tile_at = (size_t)blockIdx.z * gridDim.x + blockIdx.x;
     for (int e = threadIdx.x; e < ti.nq * HD; e += blockDim.x) {
         const int i = e / HD, r = e % HD;
         float s = 0.f;
-        for (int sp = 0; sp < a.splits; ++sp) s += a.opart[(((size_t)blockIdx.x * a.splits + sp) * a.QT + i) * HD + r];
-        const size_t at = (size_t)(ti.t0 + i) * HD + r;
+        for (int sp = 0; sp < a.splits; ++sp) s += a.opart[((tile_at * a.splits + sp) * a.QT + i) * HD + r];
+        const size_t at = (size_t)(ti.t0 + i) * a.Hp * a.Dv + (size_t)blockIdx.z * HD + r;
         if (a.out_f32) ((float*)a.out)[at] = s; else ((T*)a.out)[at] = from_f<T>(s);
     }
 }
@@ -262,14 +267,15 @@ extern "C" long long pe_attention_headmix_scratch_floats(int n_tiles, int splits
 
 template <typename T, int NACC>
 static int hm_launch(const HeadMixArgs& a, int n_tiles, size_t smem, cudaStream_t s) {
+    const int slices = a.Hp / a.H;
     PE_TRY(cudaFuncSetAttribute(headmix_kernel<T, 0, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     PE_TRY(cudaFuncSetAttribute(headmix_kernel<T, 1, NACC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    PE_TRY(pe_launch(headmix_kernel<T, 0, 1>, dim3(n_tiles, a.splits), HM_THREADS, smem, s, a));
+    PE_TRY(pe_launch(headmix_kernel<T, 0, 1>, dim3(n_tiles, a.splits, slices), HM_THREADS, smem, s, a));
     PE_LAUNCH_CHECK();
-    PE_TRY(pe_launch(headmix_kernel<T, 1, NACC>, dim3(n_tiles, a.splits), HM_THREADS, smem, s, a));
+    PE_TRY(pe_launch(headmix_kernel<T, 1, NACC>, dim3(n_tiles, a.splits, slices), HM_THREADS, smem, s, a));
     PE_LAUNCH_CHECK();
     if (a.splits > 1) {
-        PE_TRY(pe_launch(headmix_reduce_kernel<T>, n_tiles, 256, 0, s, a));
+        PE_TRY(pe_launch(headmix_reduce_kernel<T>, dim3(n_tiles, 1, slices), 256, 0, s, a));
         PE_LAUNCH_CHECK();
     }
     return 0;
@@ -280,9 +286,12 @@ extern "C" int pe_attention_headmix(const void* q, int q_stride, void* out, cons
                                     const int* tiles, int n_runs, int tile_tokens, int T, int H, int G, int D, int Dv,
                                     int window, float scale, const void* sink, int sink_dtype, const void* mix, int mix_dtype,
                                     int QT, int splits, float* scratch, const float* slopes, int keep_first, int v_ld, int v_share,
-                                    int out_f32, void* stream) {
+                                    int out_f32, int slices, void* stream) {
     if (T <= 0) return 0;
-    if (v_share < 1 || G % v_share) return PE_ERR_UNSUPPORTED;
+    if (H <= 0 || G <= 0 || H % G || v_share < 1 || slices < 1 || G % slices || (slices > 1 && mix) || (G / slices) % v_share || slices > 65535)
+        return PE_ERR_UNSUPPORTED;
+    const int Hp = H, Gp = G;
+    H /= slices; G /= slices;
     if (v_ld <= 0) v_ld = Dv;
     if (v_ld < Dv || keep_first < 0) return PE_ERR_UNSUPPORTED;
     if (H <= 0 || G <= 0 || H % G || QT < 1 || splits < 1 || splits > 65535 || (tiles && (tile_tokens % QT || n_runs <= 0)))
@@ -293,7 +302,7 @@ extern "C" int pe_attention_headmix(const void* q, int q_stride, void* out, cons
     const int n_tiles = tiles ? n_runs * (tile_tokens / QT) : T;
     HeadMixArgs a = {q, q_stride, k_pool, v_pool, table, table_stride, tok_pos, tok_row, tiles, tile_tokens, H, G, D, Dv, window,
                      scale, sink, sink_dtype, mix, mix_dtype, QT, splits, slopes, keep_first, v_ld, scratch,
-                     scratch + (size_t)n_tiles * splits * QT * H * 2, out, v_share, out_f32};
+                     scratch + (size_t)n_tiles * slices * splits * QT * H * 2, out, Hp, Gp, v_share, out_f32};
     cudaStream_t s = (cudaStream_t)stream;
     const int nacc = (int)(((size_t)H * QT * Dv + HM_THREADS - 1) / HM_THREADS);
     if (dtype == PE_F32) {

@@ -967,22 +967,28 @@ def attention_headmix(q: torch.Tensor, q_stride: int, n_heads: int, n_kv: int, h
                                                window or 0, float(scale), _ptr(sink), _ptr(mix), splits, ws.data_ptr(), stream_ptr()),
                   "attention_headmix_mma", 1 if splits == 1 else 3)
             return out
-    qt = lib.pe_attention_headmix_tile(n_heads, n_kv, head_dim, v_head_dim, 0 if mix is None else 1, 1 if tiles is None else 16)
+    # heads that do not all fit a block (without mixing they need not): slices of neighbouring key heads, each with its value heads whole
+    for slices in range(1, 1 + (n_kv // v_share if mix is None else 1)):
+        if n_kv % slices or (n_kv // slices) % v_share:
+            continue
+        qt = lib.pe_attention_headmix_tile(n_heads // slices, n_kv // slices, head_dim, v_head_dim, 0 if mix is None else 1, 1 if tiles is None else 16)
+        if qt > 0:
+            break
     if qt <= 0:
-        raise KernelError(f"attention with {n_heads} heads of size {head_dim}/{v_head_dim} is not taken: heads x value size "
-                          f"may be 16384 at most")
+        raise KernelError(f"attention with {n_heads} heads of size {head_dim}/{v_head_dim} is not taken: the heads of a key/value head times the "
+                          f"value size (with mixing: all heads) may be 16384 at most")
     n_tiles = T if tiles is None else n_runs * (PREFILL_TILE // qt)
     # few tiles with many keys (single tokens with long contexts): the keys are cut into ranges so that the GPU is filled
     splits = 1
     if n_tiles < 296:
         splits = max(1, min(296 // max(n_tiles, 1), (ctx.max_context + 255) // 256, 64))
-    ws = scratch("attention_headmix", 4 * lib.pe_attention_headmix_scratch_floats(n_tiles, splits, qt, n_heads, v_head_dim), q.device)
+    ws = scratch("attention_headmix", 4 * lib.pe_attention_headmix_scratch_floats(n_tiles * slices, splits, qt, n_heads // slices, v_head_dim), q.device)
     check(lib.pe_attention_headmix(q.data_ptr(), q_stride, out.data_ptr(), k_pool.data_ptr(), v_pool.data_ptr(), _code(q, "q"),
                                    block_table.data_ptr(), table_stride, tok_pos.data_ptr(), tok_row.data_ptr(), _ptr(tiles),
                                    n_runs, PREFILL_TILE, T, n_heads, n_kv, head_dim, v_head_dim, window or 0, float(scale),
                                    _ptr(sink), 0 if sink is None else _code(sink, "sink"), _ptr(mix),
                                    0 if mix is None else _code(mix, "mix"), qt, splits, ws.data_ptr(), _ptr(slopes), keep_first, v_ld,
-                                   v_share, 1 if out.dtype == torch.float32 and q.dtype != torch.float32 else 0, stream_ptr()),
+                                   v_share, 1 if out.dtype == torch.float32 and q.dtype != torch.float32 else 0, slices, stream_ptr()),
           "attention_headmix", 2 + (splits > 1))
     return out
 
@@ -1651,12 +1657,51 @@ def map_difference(maps: torch.Tensor, n_heads: int, n_kv: int, v_head_dim: int,
                                      _code(out, "out"), out.shape[1], out_col, stream_ptr()), "map_difference")
 
 
+# Which kernels run differential attention in bfloat16: "1" the tcgen05 kernel for prompts and the cluster kernel for single tokens where
+# they take the sizes; "mma" the mma.sync kernel for prompts too; "0" the float32-FMA kernel that takes any size (the tests run all).
+DIFF_ATTENTION = os.environ.get("PICO_ENGINE_DIFF_ATTENTION", "1")
+
+
+def _step_tiles(ctx, tile: int, device) -> torch.Tensor:
+    """The step's tokens in runs of at most ``tile``, made once a step."""
+    name = "prefill_tiles_128" if tile == PREFILL_TILE_TCGEN05 else "prefill_tiles"
+    tiles = ctx.scratch.get(name)
+    if tiles is None:
+        tiles = ctx.scratch[name] = prefill_tiles(ctx.lens, ctx.starts, device, tile)
+    return tiles
+
+
 def attention_maps(q: torch.Tensor, n_heads: int, n_kv: int, head_dim: int, v_head_dim: int, k_pool: torch.Tensor, v_pool: torch.Tensor,
                    block_table: torch.Tensor, table_stride: int, tok_pos: torch.Tensor, tok_row: torch.Tensor, window: Optional[int], scale: float,
                    lam: float, eps: float, out_scale: float, out: torch.Tensor, out_col: int, ctx) -> None:
     """Differential attention of the step's tokens over the cache into columns ``out_col`` .. of out [T, ld] (a head = ``v_head_dim`` columns,
     heads in their order).  The rows of ``q`` [T, ld2] begin with the queries laid out key/value head by key/value head as [map 1 of its
     heads | map 2 of its heads]; ``k_pool`` has 2 n_kv heads (key/value head g's maps at 2g and 2g + 1), ``v_pool`` n_kv."""
+    from .library import joined
+    T = tok_pos.shape[0]
+    _need(q, "q"); _need(k_pool, "k_pool", q.dtype); _need(v_pool, "v_pool", q.dtype); _need(out, "out", q.dtype)
+    _need(block_table, "block_table", torch.int32); _need(tok_pos, "tok_pos", torch.int32, (T,)); _need(tok_row, "tok_row", torch.int32, (T,))
+    if tuple(k_pool.shape[1:]) != (2 * n_kv, PAGE, head_dim) or tuple(v_pool.shape[1:]) != (n_kv, PAGE, v_head_dim):
+        raise KernelError("cache pools do not have the heads and head sizes of this attention")
+    if out.shape[0] != T or q.shape[0] != T or out_col + n_heads * v_head_dim > out.shape[1] or 2 * n_heads * head_dim > q.shape[1]:
+        raise KernelError("queries or heads do not fit their rows")
+    if q.dtype == torch.bfloat16 and DIFF_ATTENTION in ("1", "mma"):
+        lib = joined()
+        if (DIFF_ATTENTION == "1" and not ctx.one_token_each and scale > 0 and lib.pe_attention_diff_tcgen05_takes(n_heads, n_kv, head_dim, v_head_dim)
+                and q.shape[1] % 8 == 0 and out.shape[1] % 8 == 0 and out_col % 8 == 0):
+            tiles = _step_tiles(ctx, PREFILL_TILE_TCGEN05, q.device)
+            check(lib.pe_attention_diff_tcgen05(q.data_ptr(), q.shape[1], out.data_ptr(), out.shape[1], out_col, k_pool.data_ptr(), v_pool.data_ptr(),
+                                                k_pool.shape[0], block_table.data_ptr(), table_stride, tiles.data_ptr(), tiles.shape[0], T, n_heads,
+                                                n_kv, head_dim, v_head_dim, window or 0, float(scale), float(lam), float(eps), float(out_scale),
+                                                status_ptr(q.device), stream_ptr()), "attention_diff_tcgen05")
+            return
+        if (lib.pe_attention_diff_takes(n_heads, n_kv, head_dim, v_head_dim) and q.shape[1] % 2 == 0 and out.shape[1] % 2 == 0 and out_col % 2 == 0):
+            tiles = None if ctx.one_token_each else _step_tiles(ctx, PREFILL_TILE, q.device)
+            check(lib.pe_attention_diff(q.data_ptr(), q.shape[1], out.data_ptr(), out.shape[1], out_col, k_pool.data_ptr(), v_pool.data_ptr(),
+                                        block_table.data_ptr(), table_stride, tok_pos.data_ptr(), tok_row.data_ptr(), _ptr(tiles),
+                                        0 if tiles is None else tiles.shape[0], T, n_heads, n_kv, head_dim, v_head_dim, window or 0, float(scale),
+                                        float(lam), float(eps), float(out_scale), int(ctx.max_context), stream_ptr()), "attention_diff")
+            return
     maps = attention_headmix(q, q.shape[1], 2 * n_heads, 2 * n_kv, head_dim, v_head_dim, k_pool, v_pool, block_table, table_stride, tok_pos, tok_row,
                              window, scale, None, None, ctx, v_share=2, out_dtype=torch.float32)
     map_difference(maps, n_heads, n_kv, v_head_dim, lam, eps, out_scale, out, out_col)

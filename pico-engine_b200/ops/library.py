@@ -30,7 +30,7 @@ GATED_SOURCES = ("linear_attention.cu", "linear_attention_tiles.cu", "gated_ops.
 STATE_SOURCES = ("state_space.cu", "latent_ops.cu")
 # The kernels of sublayers that read the same rows and share their first and last product, of heads with several maps, and of routers
 # that read normed rows.
-JOINED_SOURCES = ("joined_ops.cu",)
+JOINED_SOURCES = ("joined_ops.cu", "attention_diff.cu", "attention_diff_tcgen05.cu")
 HEAD_DIM_SOURCES = ("attention_decode.cu", "attention_prefill.cu", "attention_prefill_tcgen05.cu")      # compiled per head size
 
 _SIGNATURES = {
@@ -67,7 +67,7 @@ _MIXER_SIGNATURES = {
     "pe_conv_state_update": [P, P, LL, P, P, P, I, I, I, P],
     "pe_dual_layernorm_conv": [P, P, I, P, I, P, I, P, P, P, I, P, I, P, I, P, P, I, LL, P, P, P, P, F, I, I, I, I, I, P],
     "pe_mingru": [P, I, P, LL, P, P, P, P, P, I, I, I, I, P, P],
-    "pe_attention_headmix": [P, I, P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, I, I, I, P, P, I, I, I, I, P],
+    "pe_attention_headmix": [P, I, P, P, P, I, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, I, P, I, I, I, P, P, I, I, I, I, I, P],
     "pe_qknorm_store": [P, I, I, I, I, I, I, P, I, P, I, F, P, P, P, P, P, I, I, P],
     "pe_attention_flashmix": [P, I, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, P, P, I, P, P, I, I, P],
     "pe_attention_headmix_mma": [P, I, P, P, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, P, I, P, P],
@@ -103,6 +103,10 @@ _STATE_SIGNATURES = {
 
 _JOINED_SIGNATURES = {
     "pe_heads_norm_store": [P, I, I, I, I, I, I, I, I, P, I, P, I, F, P, I, P, P, P, P, P, I, I, P],
+    "pe_attention_diff_takes": [I, I, I, I],
+    "pe_attention_diff": [P, I, P, I, I, P, P, P, I, P, P, P, I, I, I, I, I, I, I, F, F, F, F, I, P],
+    "pe_attention_diff_tcgen05_takes": [I, I, I, I],
+    "pe_attention_diff_tcgen05": [P, I, P, I, I, P, P, LL, P, I, P, I, I, I, I, I, I, I, F, F, F, F, P, P],
     "pe_map_difference": [P, I, I, I, I, F, F, F, P, I, I, I, P],
     "pe_side_act": [P, I, I, I, I, I, I, I, P, I, I, I, P, I, I, P],
     "pe_route_rows": [P, I, P, I, I, I, I, P, I, I, F, P, P, I, P],
