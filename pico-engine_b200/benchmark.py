@@ -132,7 +132,8 @@ def _mixing_flops(spec, tokens: int) -> float:
     if hasattr(spec, "n_kv_heads"):
         w = spec.window
         seen = sum(min(p + 1, w) if w else p + 1 for p in range(tokens))
-        return 2.0 * spec.n_heads * (spec.head_dim + getattr(spec, "v_head_dim", spec.head_dim)) * seen
+        maps = getattr(spec, "maps", 1)                    # maps a head has, each with a query and a key of its own
+        return 2.0 * maps * spec.n_heads * (spec.head_dim + getattr(spec, "v_head_dim", spec.head_dim)) * seen
     if hasattr(spec, "n_heads") and hasattr(spec, "v_head_dim"):
         return 4.0 * spec.n_heads * spec.head_dim * spec.v_head_dim * tokens
     return 0.0
@@ -145,7 +146,7 @@ def prefill_flops(engine, tokens: int) -> float:
     flops = 0.0
     for entry in model.plan.schedule:
         layer = model.layers[entry.layer]
-        for part in (layer.mixer, layer.feed_forward):
+        for part in (layer.mixer, layer.feed_forward, layer.joined):
             if part is not None:
                 flops += sum(2.0 * tokens * t.numel() for t in part.weights() if t.dim() == 2)
         if layer.mixer is not None:

@@ -158,6 +158,32 @@ SHAPES.update({
 })
 
 
+def razelorn_shape(width: int, heads: int, kv_heads: int, dim: int, ff: int, layers: int, vocab: int, window: int | None = None, experts: int = 8,
+                   top: int = 2, identity: int = 2, reuse: bool = False) -> dict:
+    """A Razelorn config.json whose heads have values of ``dim`` entries and two maps of ``dim`` / 2 (so that the four projections have the
+    sizes of a plain attention of ``heads`` heads of ``dim``), three quarters of a map rotated, and whose layers have in turn the dense
+    feed-forward and a mixture whose experts and shared expert are a quarter as wide.  ``reuse``: from the third layer on every layer
+    runs the tensors of the layer two before it."""
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim // 2, "vdim": dim, "scale": (dim // 2) ** -0.5, "diff": 0.5,
+             "rot": {"base": 500000.0, "dims": max(2, dim // 2 * 3 // 4 // 2 * 2), "scaling": {"factor": 8.0, "high": 4.0, "low": 1.0, "original": 8192}}}
+    if window is not None:
+        mixer["mask"] = {"size": window}
+    moe = {"expert": {"ff": ff // 4}, "kind": "moe", "router": {"experts": experts, "identity": identity, "top": top}, "shared": {"ff": ff // 4}}
+    out = []
+    for i in range(layers):
+        out.append({"mixer": dict(mixer), "mlp": {"ff": ff, "kind": "dense"} if i % 2 == 0 else dict(moe), "type": "attention"})
+        if reuse and i >= 2:
+            out[-1]["weights_of"] = i - 2
+    return {"architecture": "Razelorn", "embedding": {"scale": float(width) ** 0.5}, "layers": out, "norm": {"eps": 1e-6}, "vocab": vocab, "width": width}
+
+
+SHAPES.update({
+    "razelorn-tiny": razelorn_shape(64, 4, 2, 32, 160, 4, 256, window=40, experts=4, identity=1, reuse=True),
+    "razelorn-0.5b": razelorn_shape(896, 7, 1, 128, 4864, 24, 151936, window=1024),      # the widths of qwen2.5-0.5b
+    "razelorn-7b": razelorn_shape(3584, 28, 4, 128, 18944, 28, 152064, window=1024),     # the widths of qwen2.5-7b
+})
+
+
 def with_layers(d: dict, n: int) -> dict:
     """The shape with only its first ``n`` layers (a run of them that is repeated ends where they end)."""
     d = dict(d)

@@ -11,7 +11,7 @@ with its implementation in ``parts.registry``; nothing in this file has to chang
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import Optional, Tuple
+from typing import ClassVar, Optional, Tuple
 
 
 class ConfigError(ValueError):
@@ -289,6 +289,7 @@ class DifferentialAttentionSpec(PartSpec):
     k_name: str = "k"
     v_name: str = "v"
     o_name: str = "o"
+    maps: ClassVar[int] = 2
 
 
 @dataclass(frozen=True)

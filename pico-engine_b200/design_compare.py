@@ -8,11 +8,13 @@ row behind a sliding window; grouped attention with one added to the softmax den
 output gate; a clamped gated feed-forward; mixtures chosen by sigmoid scores among groups of experts; its kernels also beside Pupidra's like
 kernels) or the Lefilorn decoder (a residual of several streams; windowed attention with kept first keys and a norm over all query and all key
 rows beside rotated linear attention with a fixed decay, sharing their first and last product; a relu gated feed-forward; its kernels also
-beside Kevelorn's like kernels) and the dense Qwen2 decoder, this library's closest other model.  Random weights; prefill and decode throughput of a few layers, and
+beside Kevelorn's like kernels) or the Razelorn decoder (parallel layers with one layer norm, both sublayers on one first and one last product;
+differential attention with query/key norm per map; a relu^2 feed-forward; mixtures chosen by softmax scores with a correction, experts that
+pass their input on and a shared expert; its kernels also beside Tenusun's like kernels) and the dense Qwen2 decoder, this library's closest other model.  Random weights; prefill and decode throughput of a few layers, and
 the kernels of the new design each beside the Qwen2 kernel that does the like job, as fractions of the measured
 copy bandwidth or matrix throughput.
 
-    python -m pico_engine.design_compare [--design mebalorn|kevelorn|pupidra|tenusun|lefilorn] [--sizes s,m,l] [--tokens 2048] [--batch 8] [--context 2048] [--output FILE]
+    python -m pico_engine.design_compare [--design mebalorn|kevelorn|pupidra|tenusun|lefilorn|razelorn] [--sizes s,m,l] [--tokens 2048] [--batch 8] [--context 2048] [--output FILE]
 """
 from __future__ import annotations
 
@@ -62,10 +64,18 @@ def lefilorn_config(size: str, layers: int | None = None) -> dict:
     return lefilorn_shape(W, H, G, D, F, layers or max(L, 4), VOCAB)
 
 
+def razelorn_config(size: str, layers: int | None = None) -> dict:
+    from .config.shapes import razelorn_shape
+    W, H, G, D, F, L = SIZES[size]
+    # two maps of 64 over values of 128: the same projections as Qwen2's H heads of D; every earlier key visible, as there and in Tenusun
+    return razelorn_shape(W, H * D // 128, G * D // 128, 128, F, layers or max(L, 4), VOCAB)
+
+
 DESIGNS = {"mebalorn": mebalorn_config, "kevelorn": kevelorn_config, "pupidra": pupidra_config, "tenusun": tenusun_config,
-           "lefilorn": lefilorn_config}
-FOUR_LAYERS = ("pupidra", "tenusun", "lefilorn")
-BESIDE = {"tenusun": ("pupidra", pupidra_config), "lefilorn": ("kevelorn", lambda size: kevelorn_config(size, 4))}     # the closest other design
+           "lefilorn": lefilorn_config, "razelorn": razelorn_config}
+FOUR_LAYERS = ("pupidra", "tenusun", "lefilorn", "razelorn")
+BESIDE = {"tenusun": ("pupidra", pupidra_config), "lefilorn": ("kevelorn", lambda size: kevelorn_config(size, 4)),
+          "razelorn": ("tenusun", tenusun_config)}     # the closest other design
 
 
 def qwen2_config(size: str, layers: int | None = None) -> dict:
@@ -424,6 +434,54 @@ def lefilorn_kernel_times(eng, size: str, tokens: int, batch: int, context: int,
     B.close_sequences(eng, slots)
 
 
+def razelorn_kernel_times(eng, size: str, tokens: int, batch: int, context: int, entry) -> None:
+    """The kernels of the Razelorn parts at the sizes of this shape's layers (layers 0 and 2 with the dense feed-forward, 1 and 3 with the
+    mixture), and the vendor's first and last product of a layer."""
+    W, _, _, _, F, L = SIZES[size]
+    bf = torch.bfloat16
+    dense, moe_layer = eng.model.layers[0], eng.model.layers[1]
+    att, moe = dense.mixer, moe_layer.feed_forward
+    s = att.spec
+    H, G, D, Dv = s.n_heads, s.n_kv_heads, s.head_dim, s.v_head_dim
+
+    def calls(ctx, T, label, attention_size, times=8):
+        device_us = lambda fn: globals()["device_us"](fn, times)
+        kv = ctx.kv(0)
+        proj = torch.randn(T, dense.joined.w_in.shape[0], device="cuda").to(bf)
+        side = torch.empty(T, dense.joined.w_out.shape[1], device="cuda", dtype=bf)
+        entry(f"{label} norm per map + rotation + cache write", device_us(lambda: kernels.heads_norm_store(
+            proj, 2 * H, 2 * G, G, D, Dv, att.q_norm, att.k_norm, s.norm_eps, att.freq, att.rot_dims, ctx.tok_pos, ctx.tok_row, kv.k, kv.v, kv.table,
+            kv.stride)), nbytes=T * ((2 * H + 2 * G) * D + G * Dv) * 2 * 2)
+        entry(f"{label} attention (two maps, their difference, its norm)", device_us(lambda: kernels.attention_maps(
+            proj, H, G, D, Dv, kv.k, kv.v, kv.table, kv.stride, ctx.tok_pos, ctx.tok_row, s.window, s.scale, att.lam, s.norm_eps, s.out_scale, side, 0,
+            ctx)), **attention_size)
+        entry(f"{label} relu^2 into the last product's rows", device_us(lambda: dense.feed_forward.fill_side(
+            proj, dense.joined.cols[1], side, dense.joined.side_cols[1], None, ctx)), nbytes=T * F * 2 * 2)
+        h = torch.randn(T, W, device="cuda").to(bf)
+        wts = moe.routing(h)
+        mproj = torch.randn(T, moe_layer.joined.w_in.shape[0], device="cuda").to(bf)
+        mside = torch.empty(T, moe_layer.joined.w_out.shape[1], device="cuda", dtype=bf)
+        entry(f"{label} router + softmax over all + correction + choice", device_us(lambda: moe.routing(h)),
+              nbytes=T * (W * 2 + wts.shape[1] * 4) + moe.w_router.numel() * 2)
+        entry(f"{label} silu(gate) x up x expert weight", device_us(lambda: moe._hidden_units(
+            mproj, moe_layer.joined.cols[1], mside, moe_layer.joined.side_cols[1], wts)), nbytes=T * moe._width() * 2 * 3)
+        x, y = torch.randn(T, W, device="cuda"), torch.randn(T, W, device="cuda")
+        n = dense.mixer_norm
+        entry(f"{label} sublayers' sum + passed-on rows into the stream + next norm", device_us(lambda: kernels.add_layernorm(
+            x, y, (n.weight, n.bias, n.eps), bf, h, wts[:, -1])), nbytes=T * W * (4 * 3 + 2 * 2))
+        ids = torch.randint(0, VOCAB, (T,), device="cuda", dtype=torch.int32)
+        entry(f"{label} token rows x scale", device_us(lambda: kernels.embed(eng.model.embedding, ids, scale=eng.model.plan.embedding_scale)), nbytes=T * W * (2 + 4))
+
+    slot, ctx = _prompt_context(eng, tokens)
+    window = s.window or tokens
+    seen = sum(min(p + 1, window) for p in range(tokens))
+    calls(ctx, tokens, "prefill", dict(flops=4.0 * H * (D + Dv) * seen))
+    eng.cache.close(slot)
+    slots, ctx = _decode_context(eng, batch, context)
+    calls(ctx, batch, "decode", dict(nbytes=batch * min(context, window) * G * (2 * D + Dv) * 2), times=32)     # (short kernels: more of them a graph)
+    B.close_sequences(eng, slots)
+
+
 def kernel_times(size: str, tokens: int, batch: int, context: int, peaks: dict, design: str = "mebalorn") -> Dict[str, dict]:
     """Every kernel of the new design beside the like kernel of the Qwen2 decoder: microseconds, the bytes or
     multiply-adds it must move or do, and that as a fraction of the measured peak."""
@@ -448,11 +506,15 @@ def kernel_times(size: str, tokens: int, batch: int, context: int, peaks: dict, 
         other, other_config = BESIDE[design]
         runs.insert(1, (other + " beside", kevelorn_config(size, 3) if other == "kevelorn" else other_config(size)))
     for design, cfg in runs:
-        if design in ("pupidra", "pupidra beside", "tenusun", "lefilorn", "kevelorn beside"):
+        if design in ("pupidra", "pupidra beside", "tenusun", "tenusun beside", "lefilorn", "kevelorn beside", "razelorn"):
             eng = Engine.from_config(config_from_dict(cfg), seed=1, draw_on="cuda", dtype="bfloat16")
             eng.ensure_cache(max(tokens, batch * context) + 64 * batch, max(tokens, context), max_seqs=batch + 1)
             if design == "tenusun":
                 tenusun_kernel_times(eng, size, tokens, batch, context, entry)
+            elif design == "razelorn":
+                razelorn_kernel_times(eng, size, tokens, batch, context, entry)
+            elif design == "tenusun beside":
+                tenusun_kernel_times(eng, size, tokens, batch, context, _prefixed(entry, out, "tenusun "))
             elif design == "lefilorn":
                 lefilorn_kernel_times(eng, size, tokens, batch, context, entry)
             elif design == "pupidra":
