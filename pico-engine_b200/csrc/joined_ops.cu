@@ -11,7 +11,7 @@
 extern "C" void pe_set_pdl(int on) { pe_pdl_enabled() = on ? 1 : 0; }     // (this library's own copy of the switch)
 
 // ---------------------------------------------------------------- norm, rotation and cache write of query and key rows
-#define HN_THREADS 128
+#define HN_THREADS 256
 #define HN_MAX_D 256
 
 struct HeadsNormArgs {
@@ -24,23 +24,34 @@ struct HeadsNormArgs {
 
 __device__ __forceinline__ int hn_pow2(int v) { int p = 1; while (p < v) p <<= 1; return p; }
 
+// eight neighbouring entries of a norm weight (or ones)
+__device__ __forceinline__ void hn_weights8(const void* w, int dtype, int at, float* f) {
+    if (!w) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = 1.f;
+    } else if (dtype == PE_BF16 && !((uintptr_t)w & 15)) {
+        const uint4 r = *reinterpret_cast<const uint4*>((const bf16*)w + at);
+        const __nv_bfloat162* r2 = reinterpret_cast<const __nv_bfloat162*>(&r);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) { const float2 v = __bfloat1622float2(r2[e]); f[2 * e] = v.x; f[2 * e + 1] = v.y; }
+    } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] = load_as_f(w, dtype, at + e);
+    }
+}
+
 // VEC: bfloat16 with D, Dv and the row length multiples of 8: a head is D / 8 neighbouring lanes (padded to a power of two), a lane
 // holds eight entries; else a head is a warp and a lane holds every 32nd entry.  Normed rows meet in shared memory as float32 for the
-// rotation.  A block a token.
+// rotation.  A block a token (VEC: or gridDim.y blocks, each with its share of the heads, where the tokens are few); a pass's entries are
+// asked for before the pass in front of it, and the first one's before the angles, are worked out.
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(HN_THREADS) heads_norm_store_kernel(HeadsNormArgs a) {
     pdl_launch_dependents();
     __shared__ float s_cos[HN_MAX_D / 2], s_sin[HN_MAX_D / 2];
     __shared__ __align__(16) float s_row[HN_THREADS / 32][8 * 32];
-    pdl_wait();
-    const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int nt = blockDim.x, t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int D = a.D, half = a.rot >> 1, n_heads = a.H + a.G;
     T* row = (T*)a.proj + (size_t)t * a.ld;
-    const int pos = a.tok_pos[t], in_page = pos % PE_PAGE;
-    long long page = -1;
-    if (a.store) page = a.table[(size_t)a.tok_row[t] * a.table_stride + pos / PE_PAGE];
-    for (int i = tid; i < half; i += HN_THREADS) sincosf((float)pos * a.freq[i], &s_sin[i], &s_cos[i]);
-    __syncthreads();
     T* k_pool = (T*)a.k_pool;
     T* v_pool = (T*)a.v_pool;
     if constexpr (VEC) {
@@ -48,12 +59,31 @@ __global__ void __launch_bounds__(HN_THREADS) heads_norm_store_kernel(HeadsNormA
         const int sub = lane / P, l = lane % P;
         const bool on = l < L;
         float* buf = s_row[warp] + sub * (P * 8);
-        for (int h0 = warp * per_warp; h0 < n_heads; h0 += (HN_THREADS / 32) * per_warp) {
-            const int h = h0 + sub;
+        float qw[8], kw[8];
+        if (on) { hn_weights8(a.q_w, a.qw_dtype, l * 8, qw); hn_weights8(a.k_w, a.kw_dtype, l * 8, kw); }
+        pdl_wait();
+        const int step = (nt / 32) * per_warp * gridDim.y;
+        int h = (blockIdx.y * (nt / 32) + warp) * per_warp + sub;
+        uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+        if (on && h < n_heads) raw = *reinterpret_cast<const uint4*>(row + (size_t)h * D + l * 8);
+        const int pos = a.tok_pos[t], in_page = pos % PE_PAGE;
+        long long page = -1;
+        if (a.store) page = a.table[(size_t)a.tok_row[t] * a.table_stride + pos / PE_PAGE];
+        for (int i = tid; i < half; i += nt) sincosf((float)pos * a.freq[i], &s_sin[i], &s_cos[i]);
+        if (page >= 0) {
+            const int per = a.Dv / 8;
+            const T* v = row + (size_t)n_heads * D;
+            for (int i = tid + blockIdx.y * nt; i < a.Gv * per; i += nt * gridDim.y) {
+                const int c = i / per, d = (i % per) * 8;
+                *reinterpret_cast<uint4*>(v_pool + (((size_t)page * a.Gv + c) * PE_PAGE + in_page) * a.Dv + d) = *reinterpret_cast<const uint4*>(v + (size_t)i * 8);
+            }
+        }
+        __syncthreads();
+        for (int h_first = h - sub; h_first < n_heads; h_first += step, h += step) {      // (the whole warp together)
             const bool live = on && h < n_heads;
+            uint4 next = make_uint4(0u, 0u, 0u, 0u);
+            if (on && h + step < n_heads) next = *reinterpret_cast<const uint4*>(row + (size_t)(h + step) * D + l * 8);
             float f[8];
-            uint4 raw = make_uint4(0u, 0u, 0u, 0u);
-            if (live) raw = *reinterpret_cast<const uint4*>(row + (size_t)h * D + l * 8);
             const __nv_bfloat162* r2 = reinterpret_cast<const __nv_bfloat162*>(&raw);
             float ss = 0.f;
 #pragma unroll
@@ -63,12 +93,11 @@ __global__ void __launch_bounds__(HN_THREADS) heads_norm_store_kernel(HeadsNormA
                 ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss);
             }
             for (int o = P >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-            const void* w = h < a.H ? a.q_w : a.k_w;
-            const int wd = h < a.H ? a.qw_dtype : a.kw_dtype;
-            if (live && w) {
+            const bool query = h < a.H;
+            if (live && (query ? a.q_w : a.k_w)) {
                 const float rstd = 1.0f / sqrtf(ss / (float)D + a.eps);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) f[e] *= rstd * load_as_f(w, wd, l * 8 + e);
+                for (int e = 0; e < 8; ++e) f[e] *= rstd * (query ? qw[e] : kw[e]);
             }
             if (half) {
                 __syncwarp();
@@ -90,22 +119,21 @@ __global__ void __launch_bounds__(HN_THREADS) heads_norm_store_kernel(HeadsNormA
                 __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&raw);
 #pragma unroll
                 for (int e = 0; e < 4; ++e) o2[e] = __floats2bfloat162_rn(f[2 * e], f[2 * e + 1]);
-                if (h < a.H) *reinterpret_cast<uint4*>(row + (size_t)h * D + l * 8) = raw;
+                if (query) *reinterpret_cast<uint4*>(row + (size_t)h * D + l * 8) = raw;
                 else if (page >= 0) *reinterpret_cast<uint4*>(k_pool + (((size_t)page * a.G + (h - a.H)) * PE_PAGE + in_page) * D + l * 8) = raw;
             }
-        }
-        if (page >= 0) {
-            const int per = a.Dv / 8;
-            const T* v = row + (size_t)n_heads * D;
-            for (int i = tid; i < a.Gv * per; i += HN_THREADS) {
-                const int c = i / per, d = (i % per) * 8;
-                *reinterpret_cast<uint4*>(v_pool + (((size_t)page * a.Gv + c) * PE_PAGE + in_page) * a.Dv + d) = *reinterpret_cast<const uint4*>(v + (size_t)i * 8);
-            }
+            raw = next;
         }
         return;
     }
+    pdl_wait();
+    const int pos = a.tok_pos[t], in_page = pos % PE_PAGE;
+    long long page = -1;
+    if (a.store) page = a.table[(size_t)a.tok_row[t] * a.table_stride + pos / PE_PAGE];
+    for (int i = tid; i < half; i += nt) sincosf((float)pos * a.freq[i], &s_sin[i], &s_cos[i]);
+    __syncthreads();
     float* buf = s_row[warp];
-    for (int h = warp; h < n_heads; h += HN_THREADS / 32) {
+    for (int h = warp; h < n_heads; h += nt / 32) {
         T* v = row + (size_t)h * D;
         const void* w = h < a.H ? a.q_w : a.k_w;
         const int wd = h < a.H ? a.qw_dtype : a.kw_dtype;
@@ -127,7 +155,7 @@ __global__ void __launch_bounds__(HN_THREADS) heads_norm_store_kernel(HeadsNormA
     }
     if (page >= 0) {
         const T* v = row + (size_t)n_heads * D;
-        for (int i = tid; i < a.Gv * a.Dv; i += HN_THREADS) {
+        for (int i = tid; i < a.Gv * a.Dv; i += nt) {
             const int c = i / a.Dv, d = i % a.Dv;
             v_pool[(((size_t)page * a.Gv + c) * PE_PAGE + in_page) * a.Dv + d] = v[i];
         }
@@ -142,9 +170,14 @@ extern "C" int pe_heads_norm_store(void* proj, int dtype, int ld, int T, int H, 
     HeadsNormArgs a = {proj, ld, H, G, Gv, D, Dv, q_w, qw_dtype, k_w, kw_dtype, eps, freq, rot, tok_pos, tok_row, k_pool, v_pool, table, table_stride, store};
     cudaStream_t s = (cudaStream_t)stream;
     const bool vec = dtype == PE_BF16 && D % 8 == 0 && Dv % 8 == 0 && ld % 8 == 0 && !(((uintptr_t)proj | (uintptr_t)k_pool | (uintptr_t)v_pool) & 15);
+    // many tokens: blocks of four warps; few: eight warps and as many blocks a token as its heads take passes
+    int p = 1;
+    while (p < D / 8) p <<= 1;
+    const int per_pass = (HN_THREADS / 32) * (32 / p), passes = (H + G + per_pass - 1) / per_pass;
+    const bool few = T * passes <= 4 * 148;
     if (dtype == PE_F32) PE_TRY(pe_launch(heads_norm_store_kernel<float, false>, T, HN_THREADS, 0, s, a));
     else if (dtype != PE_BF16) return PE_ERR_UNSUPPORTED;
-    else if (vec) PE_TRY(pe_launch(heads_norm_store_kernel<bf16, true>, T, HN_THREADS, 0, s, a));
+    else if (vec) PE_TRY(pe_launch(heads_norm_store_kernel<bf16, true>, dim3(T, few ? passes : 1), few ? HN_THREADS : 128, 0, s, a));
     else PE_TRY(pe_launch(heads_norm_store_kernel<bf16, false>, T, HN_THREADS, 0, s, a));
     PE_LAUNCH_CHECK();
     return 0;
