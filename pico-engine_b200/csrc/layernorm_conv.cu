@@ -44,17 +44,6 @@ __global__ void __launch_bounds__(LN_THREADS) layernorm_kernel(const float* x, c
         o[i] = from_f<TO>((row[i] - mean) * rstd * load_as_f(w, w_dtype, i) + load_as_f(b, b_dtype, i));
 }
 
-extern "C" int pe_layernorm(const float* x, const int* rows_index, const void* w, int w_dtype, const void* b, int b_dtype,
-                            float eps, void* out, int out_dtype, int rows, int H, void* stream) {
-    if (rows <= 0) return 0;
-    cudaStream_t s = (cudaStream_t)stream;
-    if (out_dtype == PE_F32) PE_TRY(pe_launch(layernorm_kernel<float>, rows, LN_THREADS, 0, s, x, rows_index, w, w_dtype, b, b_dtype, eps, (float*)out, H));
-    else if (out_dtype == PE_BF16) PE_TRY(pe_launch(layernorm_kernel<bf16>, rows, LN_THREADS, 0, s, x, rows_index, w, w_dtype, b, b_dtype, eps, (bf16*)out, H));
-    else return PE_ERR_UNSUPPORTED;
-    PE_LAUNCH_CHECK();
-    return 0;
-}
-
 // ---------------------------------------------------------------- the convolution alone (on float32 normed rows)
 // y [T, H] float32.  Thread per (token, channel).
 template <typename TO>
@@ -469,15 +458,16 @@ extern "C" int pe_layernorm_add(float* x, const void* y, int y_dtype, const void
 // ---------------------------------------------------------------- sums into the stream, then the next layer norm
 // x[t] += y[t] (float32 or bfloat16; null: nothing) + rw[t * rw_ld] * rows[t] (in out's dtype, or float32 / bfloat16 by rows_dtype; null:
 // nothing) on the float32 stream, and with `out` also out[t] = layernorm(x[t]) * w + b of the row as it then stands.  A block a token.
+// rows_index (with neither y nor rows): out[r] is the norm of x[rows_index[r]].
 template <typename TO, int NV>
 __global__ void __launch_bounds__(LN_THREADS) add_layernorm_vec_kernel(float* x, const void* y, int y_dtype, const void* rows, int rows_dtype,
                                                                        const float* rw, int rw_ld, const void* w, int w_dtype, const void* b,
-                                                                       int b_dtype, float eps, int H, TO* out) {
+                                                                       int b_dtype, float eps, int H, TO* out, const int* rows_index) {
     pdl_launch_dependents();
     pdl_wait();
     __shared__ float scratch[33];
     const int n4 = H / 4;
-    const size_t row4 = (size_t)blockIdx.x * n4;
+    const size_t row4 = (size_t)blockIdx.x * n4, x4 = rows_index ? (size_t)rows_index[blockIdx.x] * n4 : row4;
     const float a = rows ? rw[(size_t)blockIdx.x * rw_ld] : 0.f;
     float4 xv[NV];
     float s = 0.f;
@@ -485,7 +475,7 @@ __global__ void __launch_bounds__(LN_THREADS) add_layernorm_vec_kernel(float* x,
     for (int v = 0; v < NV; ++v) {
         const int i = threadIdx.x + LN_THREADS * v;
         if (i < n4) {
-            xv[v] = ln_load4(x, row4 + i);
+            xv[v] = ln_load4(x, x4 + i);
             if (y) {
                 const float4 f = ln_load4_as_f(y, y_dtype, row4 + i);
                 xv[v].x += f.x; xv[v].y += f.y; xv[v].z += f.z; xv[v].w += f.w;
@@ -494,7 +484,7 @@ __global__ void __launch_bounds__(LN_THREADS) add_layernorm_vec_kernel(float* x,
                 const float4 f = ln_load4_as_f(rows, rows_dtype, row4 + i);
                 xv[v].x = fmaf(a, f.x, xv[v].x); xv[v].y = fmaf(a, f.y, xv[v].y); xv[v].z = fmaf(a, f.z, xv[v].z); xv[v].w = fmaf(a, f.w, xv[v].w);
             }
-            ln_store4(x, row4 + i, xv[v]);
+            if (y || a != 0.f) ln_store4(x, x4 + i, xv[v]);
             s += (xv[v].x + xv[v].y) + (xv[v].z + xv[v].w);
         }
     }
@@ -533,7 +523,7 @@ __global__ void __launch_bounds__(LN_THREADS) add_layernorm_kernel(float* x, con
         float n = x[at + i];
         if (y) n += load_as_f(y, y_dtype, at + i);
         if (a != 0.f) n = fmaf(a, load_as_f(rows, rows_dtype, at + i), n);
-        x[at + i] = n;
+        if (y || a != 0.f) x[at + i] = n;
         s += n;
     }
     if (!out) return;
@@ -545,24 +535,41 @@ __global__ void __launch_bounds__(LN_THREADS) add_layernorm_kernel(float* x, con
         out[at + i] = from_f<TO>(fmaf((x[at + i] - mean) * rstd, load_as_f(w, w_dtype, i), load_as_f(b, b_dtype, i)));
 }
 
-extern "C" int pe_add_layernorm(float* x, const void* y, int y_dtype, const void* rows, int rows_dtype, const float* rw, int rw_ld,
-                                const void* w, int w_dtype, const void* b, int b_dtype, float eps, int T, int H, void* out, int out_dtype,
-                                void* stream) {
+static int add_layernorm(float* x, const int* rows_index, const void* y, int y_dtype, const void* rows, int rows_dtype, const float* rw, int rw_ld,
+                         const void* w, int w_dtype, const void* b, int b_dtype, float eps, int T, int H, void* out, int out_dtype, void* stream) {
     if (T <= 0) return 0;
     if (H <= 0 || (out && (!w || !b)) || (rows && !rw) || (out && out_dtype != PE_BF16 && out_dtype != PE_F32)) return PE_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     const bool obf = out && out_dtype == PE_BF16;
     const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)rows | (uintptr_t)w | (uintptr_t)b | (uintptr_t)out;
 #define ALN(K, TO) PE_TRY(pe_launch(K, T, LN_THREADS, 0, s, x, y, y_dtype, rows, rows_dtype, rw, rw_ld, w, w_dtype, b, b_dtype, eps, H, (TO*)out))
-#define ALN_V(NV) do { if (obf) ALN((add_layernorm_vec_kernel<bf16, NV>), bf16); else ALN((add_layernorm_vec_kernel<float, NV>), float); } while (0)
+#define ALN_I(K, TO) PE_TRY(pe_launch(K, T, LN_THREADS, 0, s, x, y, y_dtype, rows, rows_dtype, rw, rw_ld, w, w_dtype, b, b_dtype, eps, H, (TO*)out, rows_index))
+#define ALN_V(NV) do { if (obf) ALN_I((add_layernorm_vec_kernel<bf16, NV>), bf16); else ALN_I((add_layernorm_vec_kernel<float, NV>), float); } while (0)
     if (H % 4 == 0 && H <= 4 * 4 * LN_THREADS && !(all & 15)) {
         const int nv = (H / 4 + LN_THREADS - 1) / LN_THREADS;
         if (nv <= 1) ALN_V(1); else if (nv == 2) ALN_V(2); else ALN_V(4);
+    } else if (rows_index) {
+        if (obf) PE_TRY(pe_launch(layernorm_kernel<bf16>, T, LN_THREADS, 0, s, x, rows_index, w, w_dtype, b, b_dtype, eps, (bf16*)out, H));
+        else PE_TRY(pe_launch(layernorm_kernel<float>, T, LN_THREADS, 0, s, x, rows_index, w, w_dtype, b, b_dtype, eps, (float*)out, H));
     } else {
         if (obf) ALN((add_layernorm_kernel<bf16>), bf16); else ALN((add_layernorm_kernel<float>), float);
     }
 #undef ALN_V
+#undef ALN_I
 #undef ALN
     PE_LAUNCH_CHECK();
     return 0;
+}
+
+extern "C" int pe_add_layernorm(float* x, const void* y, int y_dtype, const void* rows, int rows_dtype, const float* rw, int rw_ld,
+                                const void* w, int w_dtype, const void* b, int b_dtype, float eps, int T, int H, void* out, int out_dtype,
+                                void* stream) {
+    return add_layernorm(x, nullptr, y, y_dtype, rows, rows_dtype, rw, rw_ld, w, w_dtype, b, b_dtype, eps, T, H, out, out_dtype, stream);
+}
+
+// out[r] = layernorm(x[rows_index[r]]) (null: x[r]); x is read only.
+extern "C" int pe_layernorm(const float* x, const int* rows_index, const void* w, int w_dtype, const void* b, int b_dtype, float eps, void* out,
+                            int out_dtype, int rows, int H, void* stream) {
+    if (rows > 0 && !out) return PE_ERR_UNSUPPORTED;
+    return add_layernorm(const_cast<float*>(x), rows_index, nullptr, 0, nullptr, 0, nullptr, 0, w, w_dtype, b, b_dtype, eps, rows, H, out, out_dtype, stream);
 }

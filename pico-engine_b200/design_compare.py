@@ -459,12 +459,14 @@ def razelorn_kernel_times(eng, size: str, tokens: int, batch: int, context: int,
             proj, dense.joined.cols[1], side, dense.joined.side_cols[1], None, ctx)), nbytes=T * F * 2 * 2)
         h = torch.randn(T, W, device="cuda").to(bf)
         wts = moe.routing(h)
+        # hidden units that are read: those of the experts a token uses and the shared expert's (the others are written as zeros)
+        used = int((wts[:, :moe.spec.n_experts] > 0).sum()) * moe.spec.intermediate + T * moe.spec.shared_intermediate
         mproj = torch.randn(T, moe_layer.joined.w_in.shape[0], device="cuda").to(bf)
         mside = torch.empty(T, moe_layer.joined.w_out.shape[1], device="cuda", dtype=bf)
         entry(f"{label} router + softmax over all + correction + choice", device_us(lambda: moe.routing(h)),
               nbytes=T * (W * 2 + wts.shape[1] * 4) + moe.w_router.numel() * 2)
         entry(f"{label} silu(gate) x up x expert weight", device_us(lambda: moe._hidden_units(
-            mproj, moe_layer.joined.cols[1], mside, moe_layer.joined.side_cols[1], wts)), nbytes=T * moe._width() * 2 * 3)
+            mproj, moe_layer.joined.cols[1], mside, moe_layer.joined.side_cols[1], wts)), nbytes=T * moe._width() * 2 + 2 * 2 * used)
         x, y = torch.randn(T, W, device="cuda"), torch.randn(T, W, device="cuda")
         n = dense.mixer_norm
         entry(f"{label} sublayers' sum + passed-on rows into the stream + next norm", device_us(lambda: kernels.add_layernorm(
